@@ -8,9 +8,10 @@ from .kagorax import KagoraxConfig
 from .ruvuvik import RuvuvikConfig
 from .feruzen import FeruzenConfig
 from .nekorax import NekoraxConfig
+from .vametar import VametarConfig
 
 __all__ = [
-    "Architecture", "ConfigError", "FeruzenConfig", "KagoraxConfig", "LayerPlan", "ModelPlan", "NekoraxConfig", "PartSpec", "Qwen3Config", "RuvuvikConfig",
+    "Architecture", "ConfigError", "FeruzenConfig", "KagoraxConfig", "LayerPlan", "ModelPlan", "NekoraxConfig", "PartSpec", "Qwen3Config", "RuvuvikConfig", "VametarConfig",
     "ScheduleEntry", "architecture_of", "default_schedule", "get_architecture",
     "known_architectures", "load_config", "read_config_json", "register_architecture",
 ]

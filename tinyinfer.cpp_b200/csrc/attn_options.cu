@@ -9,10 +9,10 @@
 //    rotated) | latent of `rank` | one rotated key part of dr]: the latent is normed (RMS, a weight
 //    per element) and stored with the turned key part as ONE row of the token's page; the plain
 //    query parts and the turned query parts go out separately.
-//  * qkv_turn_store: the same columns without any norm: the first `rot` elements of every query and key
+//  * qkv_turn_store: the same columns with the norms of whole rows or none: the first `rot` elements of every query and key
 //    head are turned by the token's position (pairs of neighbours, or element i with i + rot/2), the
-//    first `v_rot` elements of every value head by frequencies of their own, keys and values go into
-//    the token's page and the queries out.  turn_rows turns the heads of finished rows by plus or minus
+//    first `v_rot` elements of every value head by frequencies of their own, values may be mixed with another layer's values of the token before
+//    that, keys and values go into the token's page and the queries out.  turn_rows turns the heads of finished rows by plus or minus
 //    their position (the way back for outputs over turned values) and multiplies by sigmoid(gate).
 //  * slice_rmsnorm: the RMS norm (a weight per element) of the first n columns of rows with a stride.
 //  * head_project: out[t, h, :] = in[t, h, :] W[h] with a matrix [n_in, n_out] per head.
@@ -62,14 +62,33 @@ __device__ __forceinline__ void fill_turn_table(float2* cs, int pairs, float pos
     }
 }
 
+// What qkv_turn_store does before it turns: an RMS norm over the whole query row and the whole key row with a
+// weight per element (or none), and values mixed with another layer's values of the same token.
+struct RowNorm { int on; float eps; const float* q_weight; const float* k_weight; };
+struct ValueMix { const float* first; int stride; float share; };
+
+__device__ __forceinline__ float row_unit(const float* row, int n, float eps, float* scratch) {
+    float ss = 0.0f;
+    for (int e = threadIdx.x; e < n; e += blockDim.x) ss = fmaf(row[e], row[e], ss);
+    return 1.0f / sqrtf(block_sum(ss, scratch) / (float)n + eps);
+}
+__device__ __forceinline__ float normed(const float* row, int e, float inv, const float* weight) {
+    return weight ? row[e] * inv * weight[e] : row[e] * inv;
+}
+__device__ __forceinline__ float mixed(const float* row, const float* first, int e, float share) {
+    return first ? (1.0f - share) * row[e] + share * first[e] : row[e];
+}
+
 template <typename TQ, typename TC>
 __global__ void __launch_bounds__(256)
-qkv_turn_store_kernel(const float* proj, int stride, const float* __restrict__ inv_freq, int rot, int halves, float mag,
+qkv_turn_store_kernel(const float* proj, int stride, const RowNorm norm, const ValueMix mix,
+                      const float* __restrict__ inv_freq, int rot, int halves, float mag,
                       const float* __restrict__ v_inv_freq, int v_rot, int v_halves,
                       const int* __restrict__ positions, const int* __restrict__ req_of_tok,
                       const int* __restrict__ block_table, int bt_stride, TC* __restrict__ pages, int num_pages,
                       int page_size, int write_kv, int num_heads, int num_kv_heads, int dk, int dv,
                       TQ* __restrict__ q_out, int* __restrict__ status) {
+    __shared__ float scratch[32];
     extern __shared__ float2 turn_table[];             // rot/2 entries for queries and keys, then v_rot/2 for values
     const int t = blockIdx.x;
     const int nq = num_heads * dk, nk = num_kv_heads * dk;
@@ -80,17 +99,22 @@ qkv_turn_store_kernel(const float* proj, int stride, const float* __restrict__ i
     float2* vcs = turn_table + (rot >> 1);
     fill_turn_table(cs, rot >> 1, pos, inv_freq, mag);
     if (write_kv) fill_turn_table(vcs, v_rot >> 1, pos, v_inv_freq, 1.0f);
+    const float* krow = row + nq;
+    const float inv_q = norm.on ? row_unit(row, nq, norm.eps, scratch) : 1.0f;
+    const float inv_k = norm.on && write_kv ? row_unit(krow, nk, norm.eps, scratch) : 1.0f;
     __syncthreads();
     const int per_head = (rot >> 1) + (dk - rot);      // items of a query or key head
     for (int e = threadIdx.x; e < num_heads * per_head; e += blockDim.x) {
         const int h = e / per_head, i = e % per_head;
         const TurnItem it = turn_item(i, rot, halves);
-        const float* x = row + (size_t)h * dk;
-        TQ* dst = q_out + (size_t)t * nq + (size_t)h * dk;
-        if (it.b < 0) { dst[it.a] = from_f32<TQ>(x[it.a]); continue; }
+        const int at = h * dk;
+        TQ* dst = q_out + (size_t)t * nq + at;
+        const float a = normed(row, at + it.a, inv_q, norm.q_weight);
+        if (it.b < 0) { dst[it.a] = from_f32<TQ>(a); continue; }
+        const float b = normed(row, at + it.b, inv_q, norm.q_weight);
         const float2 f = cs[i];
-        dst[it.a] = from_f32<TQ>(x[it.a] * f.x - x[it.b] * f.y);
-        dst[it.b] = from_f32<TQ>(x[it.b] * f.x + x[it.a] * f.y);
+        dst[it.a] = from_f32<TQ>(a * f.x - b * f.y);
+        dst[it.b] = from_f32<TQ>(b * f.x + a * f.y);
     }
     if (!write_kv) return;
     const int page = block_table[(size_t)req_of_tok[t] * bt_stride + pos_i / page_size];
@@ -100,29 +124,33 @@ qkv_turn_store_kernel(const float* proj, int stride, const float* __restrict__ i
     }
     const int slot = pos_i % page_size;
     TC* base = pages + (size_t)page * num_kv_heads * page_size * (dk + dv);
-    const float* krow = row + nq;
     for (int e = threadIdx.x; e < num_kv_heads * per_head; e += blockDim.x) {
         const int g = e / per_head, i = e % per_head;
         const TurnItem it = turn_item(i, rot, halves);
-        const float* x = krow + (size_t)g * dk;
+        const int at = g * dk;
         TC* dst = base + ((size_t)g * page_size + slot) * dk;
-        if (it.b < 0) { dst[it.a] = from_f32<TC>(x[it.a]); continue; }
+        const float a = normed(krow, at + it.a, inv_k, norm.k_weight);
+        if (it.b < 0) { dst[it.a] = from_f32<TC>(a); continue; }
+        const float b = normed(krow, at + it.b, inv_k, norm.k_weight);
         const float2 f = cs[i];
-        dst[it.a] = from_f32<TC>(x[it.a] * f.x - x[it.b] * f.y);
-        dst[it.b] = from_f32<TC>(x[it.b] * f.x + x[it.a] * f.y);
+        dst[it.a] = from_f32<TC>(a * f.x - b * f.y);
+        dst[it.b] = from_f32<TC>(b * f.x + a * f.y);
     }
     TC* vbase = base + (size_t)num_kv_heads * page_size * dk;
     const float* vrow = krow + nk;
+    const float* first = mix.first ? mix.first + (size_t)t * mix.stride : nullptr;
     const int v_per_head = (v_rot >> 1) + (dv - v_rot);
     for (int e = threadIdx.x; e < num_kv_heads * v_per_head; e += blockDim.x) {
         const int g = e / v_per_head, i = e % v_per_head;
         const TurnItem it = turn_item(i, v_rot, v_halves);
-        const float* x = vrow + (size_t)g * dv;
+        const int at = g * dv;
         TC* dst = vbase + ((size_t)g * page_size + slot) * dv;
-        if (it.b < 0) { dst[it.a] = from_f32<TC>(x[it.a]); continue; }
+        const float a = mixed(vrow, first, at + it.a, mix.share);
+        if (it.b < 0) { dst[it.a] = from_f32<TC>(a); continue; }
+        const float b = mixed(vrow, first, at + it.b, mix.share);
         const float2 f = vcs[i];
-        dst[it.a] = from_f32<TC>(x[it.a] * f.x - x[it.b] * f.y);
-        dst[it.b] = from_f32<TC>(x[it.b] * f.x + x[it.a] * f.y);
+        dst[it.a] = from_f32<TC>(a * f.x - b * f.y);
+        dst[it.b] = from_f32<TC>(b * f.x + a * f.y);
     }
 }
 
@@ -642,7 +670,9 @@ extern "C" int ti_latent_prepare(const float* qproj, int q_stride, const float* 
     return ti_check_launch("latent_prepare");
 }
 
-extern "C" int ti_qkv_turn_store(const float* proj, int stride, const float* inv_freq, int rot, int halves, float mag,
+extern "C" int ti_qkv_turn_store(const float* proj, int stride, int row_norm, float eps, const float* q_weight,
+                                 const float* k_weight, const float* mix_first, int mix_stride, float mix_share,
+                                 const float* inv_freq, int rot, int halves, float mag,
                                  const float* v_inv_freq, int v_rot, int v_halves, const int* positions,
                                  const int* req_of_tok, const int* block_table, int bt_stride, void* pages,
                                  int cache_dtype, int num_pages, int page_size, int write_kv, int num_tokens,
@@ -657,10 +687,12 @@ extern "C" int ti_qkv_turn_store(const float* proj, int stride, const float* inv
                "qkv_turn_store: a rotation needs its frequencies");
     cudaStream_t s = (cudaStream_t)stream;
     const size_t turn_smem = (size_t)(rot / 2 + v_rot / 2) * sizeof(float2);      // the token's cosines and sines
-    TI_REQUIRE(turn_smem <= 48 * 1024, "qkv_turn_store: rotated widths %d and %d", rot, v_rot);
+    const RowNorm norm{row_norm, eps, q_weight, k_weight};
+    const ValueMix mix{mix_first, mix_stride, mix_share};
+    TI_REQUIRE(turn_smem <= 47 * 1024, "qkv_turn_store: rotated widths %d and %d", rot, v_rot);
 #define CALL(TQ, TC)                                                                              \
     qkv_turn_store_kernel<TQ, TC><<<num_tokens, 256, turn_smem, s>>>(                              \
-        proj, stride, inv_freq, rot, halves, mag, v_inv_freq, v_rot, v_halves, positions, req_of_tok, \
+        proj, stride, norm, mix, inv_freq, rot, halves, mag, v_inv_freq, v_rot, v_halves, positions, req_of_tok, \
         block_table, bt_stride, (TC*)pages, num_pages, page_size, write_kv, num_heads, num_kv_heads, dk, dv, \
         (TQ*)q_out, status)
     TI_DISPATCH_QC(q_dtype, cache_dtype, CALL)

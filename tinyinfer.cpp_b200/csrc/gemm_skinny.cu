@@ -49,7 +49,7 @@ template <int NT, int ROWS, int BATCH, bool STORE_ONLY = false>
 __global__ void __launch_bounds__(WARPS * 32, BATCH == 4 && NT == 1 ? 3 : 2)
 gemm_skinny_kernel(const bf16* a, const bf16* __restrict__ w, float* __restrict__ c,
                    bf16* __restrict__ out_act, int m, int n, int k, int lda, int ldw, int ldc,
-                   int ld_act, int mode, float act_p, float act_q) {
+                   int ld_act, int mode, int glu_kind, float act_p, float act_q) {
     constexpr int MP = NT * 8;                                  // padded token count
     __shared__ float part[WARPS][ROWS][MP + 1];
     if (STORE_ONLY) mode = MODE_STORE;
@@ -157,9 +157,7 @@ gemm_skinny_kernel(const bf16* a, const bf16* __restrict__ w, float* __restrict_
                     gate += part[wp][i][tok];
                     up += part[wp][(i + 8) % ROWS][tok];
                 }
-                // act_q (the clamped gate's factor inside the sigmoid) other than 0: that activation, with the limit act_p
-                const float y = act_q != 0.0f ? glu_activation(GLU_CLAMPED, gate, up, act_p, act_q)
-                                              : gate / (1.0f + expf(-gate)) * up;
+                const float y = glu_activation(glu_kind, gate, up, act_p, act_q);   // limit act_p, factor act_q
                 if (n0 + i + 8 < n) out_act[(size_t)tok * ld_act + col] = __float2bfloat16_rn(y);
             }
         }
@@ -191,7 +189,7 @@ extern "C" int ti_gemm_skinny_supported(int m, int n, int k, int lda, int ldw) {
 // mode 0: c = a w^T; 1: c += a w^T; 2: out_act[m, n/2] = swiglu over strips of 8 gate + 8 up rows;
 // 3: out_act[m, n] = xielu(a w^T) with the activation's two factors.
 static int skinny(const void* a, const void* w, float* c, void* out_act, int m, int n, int k, int lda, int ldw,
-                  int ldc, int ld_act, int mode, float act_p, float act_q, void* stream) {
+                  int ldc, int ld_act, int mode, int glu_kind, float act_p, float act_q, void* stream) {
     if (m == 0 || n == 0) return 0;
     TI_REQUIRE(ti_gemm_skinny_supported(m, n, k, lda, ldw),
                "gemm_skinny: M=%d (1..64), K=%d (multiple of 32) or row strides %d, %d (multiples of 8) "
@@ -206,19 +204,19 @@ static int skinny(const void* a, const void* w, float* c, void* out_act, int m, 
     if (narrow)                                                                                     \
         ti_launch_pdl(gemm_skinny_kernel<NT, 8, 8>, (unsigned)((n + 7) / 8), WARPS * 32, 0, s,      \
                       (const bf16*)a, (const bf16*)w, c, (bf16*)out_act, m, n, k, lda, ldw, ldc,    \
-                      ld_act, mode, act_p, act_q);                                                                \
+                      ld_act, mode, glu_kind, act_p, act_q);                                                                \
     else if (k <= SHORT_K && mode == MODE_STORE && NT <= 2)                                         \
         ti_launch_pdl((gemm_skinny_kernel<NT <= 2 ? NT : 1, 16, 4, true>), (unsigned)((n + STRIP - 1) / STRIP), \
                       WARPS * 32, 0, s, (const bf16*)a, (const bf16*)w, c, (bf16*)out_act, m, n, k, \
-                      lda, ldw, ldc, ld_act, mode, act_p, act_q);                                   \
+                      lda, ldw, ldc, ld_act, mode, glu_kind, act_p, act_q);                                   \
     else if (k <= SHORT_K)                                                                          \
         ti_launch_pdl(gemm_skinny_kernel<NT, 16, 4>, (unsigned)((n + STRIP - 1) / STRIP),           \
                       WARPS * 32, 0, s, (const bf16*)a, (const bf16*)w, c, (bf16*)out_act, m, n, k, \
-                      lda, ldw, ldc, ld_act, mode, act_p, act_q);                                   \
+                      lda, ldw, ldc, ld_act, mode, glu_kind, act_p, act_q);                                   \
     else                                                                                            \
         ti_launch_pdl(gemm_skinny_kernel<NT, 16, 8>, (unsigned)((n + STRIP - 1) / STRIP),           \
                       WARPS * 32, 0, s, (const bf16*)a, (const bf16*)w, c, (bf16*)out_act, m, n, k, \
-                      lda, ldw, ldc, ld_act, mode, act_p, act_q)
+                      lda, ldw, ldc, ld_act, mode, glu_kind, act_p, act_q)
     if (m <= 8) { LAUNCH(1); }
     else if (m <= 16) { LAUNCH(2); }
     else if (m <= 32) { LAUNCH(4); }
@@ -230,22 +228,19 @@ static int skinny(const void* a, const void* w, float* c, void* out_act, int m, 
 extern "C" int ti_gemm_skinny(const void* a, const void* w, float* c, void* out_act, int m, int n,
                               int k, int lda, int ldw, int ldc, int ld_act, int mode, void* stream) {
     TI_REQUIRE(mode >= MODE_STORE && mode <= MODE_SWIGLU, "gemm_skinny: mode %d", mode);
-    return skinny(a, w, c, out_act, m, n, k, lda, ldw, ldc, ld_act, mode, 0.0f, 0.0f, stream);
+    return skinny(a, w, c, out_act, m, n, k, lda, ldw, ldc, ld_act, mode, GLU_SILU, 0.0f, 0.0f, stream);
 }
 
 // out_act[m, n/2] (bfloat16) = act(gate, up) over strips of 8 gate and 8 up rows of w, with the gated activation
 // `glu_kind` of glu.cuh in the epilogue.
 extern "C" int ti_gemm_skinny_glu(const void* a, const void* w, void* out_act, int m, int n, int k, int lda, int ldw,
                                   int ld_act, int glu_kind, float glu_limit, float glu_alpha, void* stream) {
-    TI_REQUIRE(glu_kind == GLU_SILU || (glu_kind == GLU_CLAMPED && glu_alpha != 0.0f),
-               "gemm_skinny_glu: activation %d (the clamped gate needs its factor)", glu_kind);
-    const bool clamped = glu_kind == GLU_CLAMPED;
-    return skinny(a, w, nullptr, out_act, m, n, k, lda, ldw, 0, ld_act, MODE_SWIGLU, clamped ? glu_limit : 0.0f,
-                  clamped ? glu_alpha : 0.0f, stream);
+    TI_REQUIRE(glu_kind >= GLU_SILU && glu_kind <= GLU_GELU_TANH, "gemm_skinny_glu: activation %d", glu_kind);
+    return skinny(a, w, nullptr, out_act, m, n, k, lda, ldw, 0, ld_act, MODE_SWIGLU, glu_kind, glu_limit, glu_alpha, stream);
 }
 
 // out_act[m, n] (bfloat16) = xielu(a w^T): act_p z^2 + z/2 for z > 0, act_q (exp(z) - 1 - z) + z/2 otherwise
 extern "C" int ti_gemm_skinny_xielu(const void* a, const void* w, void* out_act, int m, int n, int k, int lda,
                                     int ldw, int ld_act, float act_p, float act_q, void* stream) {
-    return skinny(a, w, nullptr, out_act, m, n, k, lda, ldw, 0, ld_act, MODE_XIELU, act_p, act_q, stream);
+    return skinny(a, w, nullptr, out_act, m, n, k, lda, ldw, 0, ld_act, MODE_XIELU, GLU_SILU, act_p, act_q, stream);
 }

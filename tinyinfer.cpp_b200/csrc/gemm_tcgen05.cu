@@ -525,7 +525,7 @@ extern "C" int ti_gemm_tcgen05_grouped_glu(const void* a, const void* w, void* o
                                            int lda, int ldw, int ld_act, int groups, const int* group_of_tile,
                                            const int* tiles_m_dev, int glu_kind, float glu_limit, float glu_alpha,
                                            int* status, void* stream) {
-    TI_REQUIRE(glu_kind == GLU_SILU || glu_kind == GLU_CLAMPED, "gemm_tcgen05_grouped_glu: activation %d", glu_kind);
+    TI_REQUIRE(glu_kind >= GLU_SILU && glu_kind <= GLU_GELU_TANH, "gemm_tcgen05_grouped_glu: activation %d", glu_kind);
     return gemm_tcgen05_grouped_impl(a, w, nullptr, out_act, m_max, n, k, lda, ldw, 0, ld_act, MODE_SWIGLU, groups,
                                      group_of_tile, tiles_m_dev, status, stream, GluArgs{glu_kind, glu_limit, glu_alpha});
 }
@@ -536,7 +536,7 @@ extern "C" int ti_gemm_tcgen05_glu(const void* a, const void* w, void* out_act, 
                                    int ldw, int ld_act, int glu_kind, float glu_limit, float glu_alpha, int* status,
                                    void* stream) {
     if (m == 0 || n == 0) return 0;
-    TI_REQUIRE(glu_kind == GLU_SILU || glu_kind == GLU_CLAMPED, "gemm_tcgen05_glu: activation %d", glu_kind);
+    TI_REQUIRE(glu_kind >= GLU_SILU && glu_kind <= GLU_GELU_TANH, "gemm_tcgen05_glu: activation %d", glu_kind);
     TI_REQUIRE(ti_gemm_tcgen05_supported(m, n, k, lda, ldw, 0, MODE_SWIGLU),
                "gemm_tcgen05_glu: K=%d and the row strides %d, %d must be multiples of 8, N=%d a multiple of 16", k, lda,
                ldw, n);

@@ -1,13 +1,25 @@
-// Gated activations of a feed-forward, y = act(gate, up), shared by the row-wise kernel and the
+// A sum that passes a gate, and gated activations of a feed-forward, y = act(gate, up), shared by the row-wise kernel and the
 // epilogues of the experts' products.
 //   GLU_SILU      silu(g) * u
 //   GLU_CLAMPED   g = min(g, limit), u = clamp(u, -limit, limit), y = g * sigmoid(alpha * g) * (u + 1)
+//   GLU_GELU_TANH gelu(g) * u, the tanh form of gelu
 #pragma once
 
-enum { GLU_SILU = 0, GLU_CLAMPED = 1 };
+enum { GLU_SILU = 0, GLU_CLAMPED = 1, GLU_GELU_TANH = 2 };
 
 // What an epilogue needs to know of the activation; kind GLU_SILU ignores the rest.
 struct GluArgs { int kind; float limit, alpha; };
+
+// A sublayer's result y on its way into the residual x: x + scale sigmoid(g) y
+__device__ __forceinline__ float gated_sum(float x, float y, float g, float scale) {
+    return fmaf(scale / (1.0f + expf(-g)), y, x);
+}
+
+// gelu(z) = z/2 (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))
+__device__ __forceinline__ float gelu_tanh(float z) {
+    const float inner = 0.7978845608028654f * fmaf(0.044715f * z * z, z, z);
+    return 0.5f * z * (1.0f + tanhf(inner));
+}
 
 __device__ __forceinline__ float glu_activation(int kind, float g, float u, float limit, float alpha) {
     if (kind == GLU_CLAMPED) {
@@ -15,5 +27,6 @@ __device__ __forceinline__ float glu_activation(int kind, float g, float u, floa
         u = fminf(fmaxf(u, -limit), limit);
         return g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
     }
+    if (kind == GLU_GELU_TANH) return gelu_tanh(g) * u;
     return g / (1.0f + expf(-g)) * u;
 }

@@ -190,10 +190,6 @@ class Engine:
         return logits
 
     def forward(self, batch: StepBatch) -> torch.Tensor:
-        views = {}
-        for entry in self.plan.schedule:
-            key = (entry.cache_slot, entry.writes_cache)
-            if key not in views:
-                views[key] = self.cache.view(entry.cache_slot, entry.writes_cache,
-                                             batch.block_tables, batch.state_slots)
+        views = {(slot, writes): self.cache.view(slot, writes, batch.block_tables, batch.state_slots)
+                 for slot, writes in self.model.cache_keys()}
         return self.model.forward(self.ops, batch, views)

@@ -33,7 +33,9 @@ LIBRARIES = {
     "mixers": ["common.cu", "attn_options.cu", "wkv.cu"],
     "bf16_mixers": ["common.cu", "attn_options_tc.cu"],
     # recurrent mixers with a matrix state
-    "state": ["common.cu", "matrix_state.cu"],
+    "state": ["common.cu", "matrix_state.cu", "matrix_state_decayed.cu"],
+    # recurrences per channel and the gates and decays in front of them
+    "channels": ["common.cu", "channel_recurrence.cu"],
     # short convolutions over time, norms in groups and without statistics, depth sums, gated activations
     "rows": ["common.cu", "state_rows.cu"],
 }

@@ -11,7 +11,7 @@ pack_linear(w) -> w'                         a product's weight in the layout th
 pack_gate_up(gate, up) -> w'                 the stacked gate/up weight
 embed(table, token_ids, out)                 out[t] = float32(table[token_ids[t]])
 rmsnorm(x, weight, eps, out, rows=None)      out[r] = norm(x[rows[r]] or x[r]), rounded to out.dtype
-linear(a, w, out, accumulate=False)          out (+)= a @ w.T in float32
+linear(a, w, out, accumulate=False)          out (+)= a @ w.T in float32 (or through a gate into a residual)
 linear_xielu(h, w, ap, aq, out)              out = xielu(h @ w.T), one launch for few rows
 glu_ffn(h, w_gate_up, w_down, residual, ...) residual += act(gate, up) @ w_down.T with a gated activation
 gate_up_swiglu(h, w, out)                    out = silu(h @ gate.T) * (h @ up.T)
@@ -486,9 +486,14 @@ class CudaOps(MixerOps, StateOps):
         product back and run it in one launch with a norm of ``out`` and a feed-forward into ``out``
         that follow immediately; any other operation of the kernel set, ``stream()`` and
         ``flush()`` launch it first.  The caller must not touch ``a`` or ``out`` by other means
-        until then."""
+        until then.  ``out`` may be a ``parts.base.GatedSum`` (with ``accumulate``): the product then
+        passes that gate on its way into the residual."""
         if self._pending is not None or self._pending_runs is not None:
             self.flush()
+        if not isinstance(out, torch.Tensor):
+            _need(accumulate, "linear: a gated sum adds to its residual")
+            self._linear_gated_sum(a, w, out)
+            return
         m, k = a.shape
         n = w.shape[0]
         if (may_defer and accumulate and self.fuse_decode_tail and self.fuse_decode_ffn and m <= 16 and n <= 1024
@@ -519,6 +524,12 @@ class CudaOps(MixerOps, StateOps):
             a.data_ptr(), _code(a, "linear"), w.data_ptr(), _code(w, "linear"), out.data_ptr(),
             m, n, k, a.stride(0), w.stride(0), out.stride(0), int(bool(accumulate)),
             self._stream()))
+
+    def _linear_gated_sum(self, a, w, target):
+        """``x += scale * sigmoid(gate + bias) * (a @ w.T)`` for a ``parts.base.GatedSum``."""
+        y = torch.empty((a.shape[0], w.shape[0]), dtype=torch.float32, device=a.device)
+        self.linear(a, w, y)
+        self.gated_add(y, target)
 
     def gate_up_swiglu(self, h, w_gate_up, out):
         inter = out.shape[1]
@@ -574,7 +585,7 @@ class CudaOps(MixerOps, StateOps):
         inter = w_down.shape[1]
         interleaved = bool(getattr(w_gate_up, "_ti_interleaved", False))
         y = torch.empty((m, inter), dtype=h.dtype, device=h.device)
-        if (interleaved and h.dtype == torch.bfloat16 and w_gate_up.dtype == torch.bfloat16 and float(alpha) != 0.0
+        if (interleaved and h.dtype == torch.bfloat16 and w_gate_up.dtype == torch.bfloat16
                 and h.data_ptr() % 16 == 0
                 and self.bf16.ti_gemm_skinny_supported(m, 2 * inter, k, h.stride(0), w_gate_up.stride(0))):
             # few rows: the activation in the epilogue of the product that streams the weights once

@@ -10,7 +10,7 @@ qk_rownorm_rope_store(proj, ...)     norm over the whole query row and the whole
                                      of neighbouring pairs, keys/values into pages, queries out
 latent_prepare(proj, ...)            normed latent + turned key part as one cached row; plain
                                      and turned query parts out
-qkv_turn_store(proj, ...)            no norm: queries and keys turned, values turned by frequencies of
+qkv_turn_store(proj, ...)            norms of whole rows or none, queries and keys turned, values mixed with another layer's, values turned by frequencies of
                                      their own, keys/values into pages, queries out
 slice_rmsnorm(x, weight, eps, out)   RMS norm of a column slice of a product
 turn_rows(x, step, rotation, ...)    finished rows' heads turned by plus or minus their position, times
@@ -85,7 +85,7 @@ class MixerOps:
                                                    _i, _i, _i, _i, _i, _i, _i, _i, _vp, _i, _vp, _vp]
             b.ti_latent_prepare.argtypes = [_vp, _i, _vp, _i, _vp, _f, _vp, _f, _vp, _vp, _vp, _i, _vp, _i, _i, _i, _i, _i,
                                             _i, _i, _i, _vp, _vp, _i, _vp, _vp]
-            b.ti_qkv_turn_store.argtypes = [_vp, _i, _vp, _i, _i, _f, _vp, _i, _i, _vp, _vp, _vp, _i, _vp, _i, _i, _i,
+            b.ti_qkv_turn_store.argtypes = [_vp, _i, _i, _f, _vp, _vp, _vp, _i, _f, _vp, _i, _i, _f, _vp, _i, _i, _vp, _vp, _vp, _i, _vp, _i, _i, _i,
                                             _i, _i, _i, _i, _i, _i, _vp, _i, _vp, _vp]
             b.ti_slice_rmsnorm.argtypes = [_vp, _i, _i, _i, _vp, _f, _vp, _i, _vp]
             b.ti_turn_rows.argtypes = [_vp, _i, _vp, _vp, _i, _i, _f, _vp, _i, _i, _i, _i, _vp, _vp]
@@ -195,8 +195,12 @@ class MixerOps:
 
     _LAYOUTS = {"interleaved": 0, "neox": 1}
 
-    def qkv_turn_store(self, proj, rotation, v_rotation, step, cache, q_out, num_heads, num_kv_heads, dk, dv):
-        """From the float32 rows ``proj`` (columns: queries, keys, values): no norm; the first
+    def qkv_turn_store(self, proj, rotation, v_rotation, step, cache, q_out, num_heads, num_kv_heads, dk, dv,
+                       row_norm=None, value_mix=None):
+        """From the float32 rows ``proj`` (columns: queries, keys, values): with ``row_norm = (q_weight,
+        k_weight, eps)`` the whole query row and the whole key row are RMS-normed (weights per column, or
+        None), without it nothing is; with ``value_mix = (first, share)`` the values become ``(1 - share) v +
+        share first`` (``first`` float32 rows like the values; a column slice is fine).  Then the first
         ``rotation.rotary_dim`` elements of every query and key head are turned by the token's
         position (kind ``interleaved``: neighbouring pairs; ``neox``: element ``i`` with ``i +
         rotary_dim / 2``; ``none``), the first ``v_rotation.rotary_dim`` elements of every value
@@ -221,8 +225,16 @@ class MixerOps:
                    "qkv_turn_store: page layout")
         self._must(bt.dtype == torch.int32 and bt.stride(1) == 1, "qkv_turn_store: block table int32")
         self._must(q_out.is_contiguous() and tuple(q_out.shape) == (t, nq), "qkv_turn_store: q_out")
+        q_weight, k_weight, eps = row_norm if row_norm is not None else (None, None, 0.0)
+        for w, n in ((q_weight, nq), (k_weight, nk)):
+            self._must(w is None or (w.dtype == torch.float32 and w.is_contiguous() and w.shape[0] == n),
+                       "qkv_turn_store: a norm weight must be float32, one value per column")
+        first, share = value_mix if value_mix is not None else (None, 0.0)
+        self._must(first is None or (first.dtype == torch.float32 and first.stride(1) == 1 and tuple(first.shape) == (t, nv)),
+                   "qkv_turn_store: the values to mix in must be float32 rows of this layer's values' size")
         self._mx(self.mixers.ti_qkv_turn_store(
-            proj.data_ptr(), proj.stride(0), rots[0][2], rots[0][0], rots[0][1], rots[0][3], rots[1][2], rots[1][0],
+            proj.data_ptr(), proj.stride(0), int(row_norm is not None), float(eps), _ptr(q_weight), _ptr(k_weight),
+            _ptr(first), first.stride(0) if first is not None else 0, float(share), rots[0][2], rots[0][0], rots[0][1], rots[0][3], rots[1][2], rots[1][0],
             rots[1][1], step.positions.data_ptr(), step.req_of_tok.data_ptr(), bt.data_ptr(), bt.stride(0),
             pages.data_ptr(), _CODE[pages.dtype], pages.shape[0], cache.page_size, int(bool(cache.writes)), t,
             num_heads, num_kv_heads, dk, dv, q_out.data_ptr(), _CODE[q_out.dtype], self.status.data_ptr(),

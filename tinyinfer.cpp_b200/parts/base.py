@@ -16,7 +16,8 @@ mixer     ``cache_spec()``: what it keeps per request (``PagedKVSpec``, ``FixedS
           None); ``forward(ops, h, residual, step, cache)``: adds its output to ``residual``.
 ffn       ``forward(ops, h, residual, step)``: adds its output to ``residual``.
 block     arrangement of the four parts of a layer: ``forward(ops, x, step, cache)``.
-embedding ``forward(ops, token_ids, out)``;  head ``forward(ops, h) -> logits``.
+embedding ``forward(ops, token_ids, out)``;  head ``forward(ops, h) -> logits``.  An embedding that
+          keeps something per request (``cache_spec()``) gets the step and its view as well.
 junction  ``forward(ops, x, x0, index, step)``: renews the residual stream ``x`` in place from itself
           and the embedding output ``x0`` where the schedule enters pass ``index`` of a run of layers.
 
@@ -86,8 +87,27 @@ class CompositeSpec:
         return out
 
 
+@dataclass(frozen=True)
+class GatedSum:
+    """Where a sublayer's last product lands when its result passes a gate on the way into the
+    residual stream: ``x += scale * sigmoid(gate + bias) * result``, element by element.  ``gate`` is
+    float32 ``[T, width]``, ``bias`` float32 ``[width]``.  ``ops.linear(a, w, target, accumulate=True)``
+    takes it in the place of a float32 residual."""
+    x: torch.Tensor
+    gate: torch.Tensor
+    bias: torch.Tensor
+    scale: float
+
+    @property
+    def shape(self):
+        return self.x.shape
+
+
 class Part:
     category = ""
+    # a mixer or feed-forward that touches its residual by one closing ``ops.linear(..., accumulate=True)``
+    # alone: a block may then hand it a ``GatedSum``
+    ends_in_linear = False
 
     def weight_specs(self) -> dict[str, WeightSpec]:
         return {}

@@ -6,6 +6,10 @@ mixer's and the feed-forward's last product.  A layer without a feed-forward sto
 
 ``parallel``: ``h = norm(x)``, then ``x += mixer(h)`` and ``x += ffn(h)``.
 
+``gated_prenorm``: ``prenorm`` whose sublayers' results pass a sigmoid gate on their way into the
+residual stream, ``x += m sigmoid(Wg h + bg) * sublayer(h)``, with an optional shift of the mixer's
+input towards the token before.
+
 ``sandwich``: a norm before and behind each sublayer, ``x += norm1b(mixer(norm1(x)))`` then
 ``x += norm2b(ffn(norm2(x)))``.
 
@@ -17,7 +21,8 @@ from __future__ import annotations
 
 import torch
 
-from .base import MATRIX, NORM_WEIGHT, CompositeSpec, FixedStateSpec, Part, WeightSpec, as_float32, register_part
+from .base import (MATRIX, NORM_WEIGHT, NORM_ZERO, CompositeSpec, FixedStateSpec, GatedSum, Part, WeightSpec, as_float32,
+                   register_part)
 
 
 class PreNormBlock(Part):
@@ -33,6 +38,72 @@ class PreNormBlock(Part):
         self.mixer.forward(ops, self.mixer_norm.forward(ops, x, step.act_dtype), x, step, cache)
         if self.ffn is not None:
             self.ffn.forward(ops, self.ffn_norm.forward(ops, x, step.act_dtype), x, step)
+
+
+class GatedPreNormBlock(Part):
+    """Pre-norm with a gate and a factor on what each sublayer adds:
+
+        h = norm1(x);   x += m sigmoid(Wg1 h + b1) * mixer(s(h))
+        h = norm2(x);   x += m sigmoid(Wg2 h + b2) * ffn(h)           (where the layer has one)
+
+    element by element, with ``m`` = ``multiplier`` (tensors ``rg1``, ``rg1.b``, ``rg2``, ``rg2.b``).
+    ``token_shift``: the mixer reads ``s(h)_t = h_t + (h_(t-1) - h_t) shift`` (tensor ``shift``, zeros in
+    front of a sequence's first token) and the request keeps its last ``h`` in float32; the gate
+    reads ``h`` itself.  What the request keeps is a composite: that row under ``shift``, the mixer's
+    own cache under ``mixer``."""
+    category = "block"
+
+    def __init__(self, mixer, mixer_norm, ffn=None, ffn_norm=None, hidden_size: int = 0, multiplier: float = 1.0,
+                 token_shift: bool = True):
+        if (ffn is None) != (ffn_norm is None):
+            raise ValueError("a feed-forward and its norm come together")
+        self.mixer, self.ffn, self.mixer_norm, self.ffn_norm = mixer, ffn, mixer_norm, ffn_norm
+        self.hidden_size, self.multiplier, self.token_shift = int(hidden_size), float(multiplier), bool(token_shift)
+        self.shift = None
+        self.gates = []                      # (matrix, bias) of the mixer's and the feed-forward's gate
+
+    def weight_specs(self):
+        n = self.hidden_size
+        specs = {"shift": WeightSpec((n,), NORM_ZERO)} if self.token_shift else {}
+        for name in ("rg1", "rg2") if self.ffn is not None else ("rg1",):
+            specs.update({name: WeightSpec((n, n), MATRIX), name + ".b": WeightSpec((n,), NORM_ZERO)})
+        return specs
+
+    def load_weights(self, tensors, ops):
+        if self.token_shift:
+            self.shift = as_float32(tensors["shift"]).contiguous()
+        self.gates = [(ops.pack_linear(tensors[name]), as_float32(tensors[name + ".b"]).contiguous())
+                      for name in (("rg1", "rg2") if self.ffn is not None else ("rg1",))]
+
+    def cache_spec(self):
+        items = [("mixer", self.mixer.cache_spec())]
+        if self.token_shift:
+            items.insert(0, ("shift", FixedStateSpec((self.hidden_size,), torch.float32)))
+        return CompositeSpec(tuple(items))
+
+    def _add(self, ops, part, run, h, x, gate):
+        """``x += m sigmoid(Wg h + b) * part(.)``; ``run(target)`` lets the part add its result to ``target``."""
+        w, bias = gate
+        g = torch.empty_like(x)
+        ops.linear(h, w, g)
+        target = GatedSum(x, g, bias, self.multiplier)
+        if part.ends_in_linear:
+            run(target)
+        else:
+            y = torch.zeros_like(x)
+            run(y)
+            ops.flush()
+            ops.gated_add(y, target)
+
+    def forward(self, ops, x, step, cache):
+        if self.token_shift:
+            h, s = self.mixer_norm.forward_shifted(ops, x, self.shift, step, cache["shift"], step.act_dtype)
+        else:
+            h = s = self.mixer_norm.forward(ops, x, step.act_dtype)
+        self._add(ops, self.mixer, lambda y: self.mixer.forward(ops, s, y, step, cache.child("mixer")), h, x, self.gates[0])
+        if self.ffn is not None:
+            h = self.ffn_norm.forward(ops, x, step.act_dtype)
+            self._add(ops, self.ffn, lambda y: self.ffn.forward(ops, h, y, step), h, x, self.gates[1])
 
 
 class ParallelBlock(Part):
@@ -161,6 +232,7 @@ class OutputNormBlock(Part):
 
 
 register_part("block", "prenorm", PreNormBlock)
+register_part("block", "gated_prenorm", GatedPreNormBlock)
 register_part("block", "output_norm", OutputNormBlock)
 register_part("block", "sandwich", SandwichBlock)
 register_part("block", "parallel", ParallelBlock)

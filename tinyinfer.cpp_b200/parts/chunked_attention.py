@@ -16,6 +16,10 @@ For token ``i`` and query head ``a`` (kv head ``a // (heads / kv_heads)``):
 ``softcap`` None; ``head_temperature``, ``head_gate`` False), and ``norm_per_head`` norms every
 query and key head by itself with one weight of ``head_dim`` elements, so other designs can use the
 part: with everything off it is plain causal grouped-query attention with a query/key norm.
+
+``value_mix`` ties the values of several layers together: the layer with ``"source"`` leaves its values
+``v1`` (float32, in the step's scratch), and a later layer with ``"mix"`` caches ``(1 - l) v + l v1`` of
+the same token (``l`` the number in the tensor ``vmix``).
 """
 from __future__ import annotations
 
@@ -24,16 +28,20 @@ from typing import Optional
 import torch
 
 from ..config.plan import PartSpec
-from .base import MATRIX, NORM_WEIGHT, PagedKVSpec, Part, WeightSpec, as_float32, build_part, register_part
+from .base import MATRIX, NORM_WEIGHT, NORM_ZERO, PagedKVSpec, Part, WeightSpec, as_float32, build_part, register_part
 
 
 class ChunkedAttention(Part):
     category = "mixer"
+    ends_in_linear = True
 
     def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, head_dim: int, v_head_dim: int,
                  scale: float, qk_norm_eps: float, position: PartSpec, chunk: Optional[int] = None,
                  window: Optional[int] = None, softcap: Optional[float] = None,
-                 head_temperature: bool = True, head_gate: bool = True, norm_per_head: bool = False):
+                 head_temperature: bool = True, head_gate: bool = True, norm_per_head: bool = False,
+                 value_mix: Optional[str] = None):
+        if value_mix not in (None, "source", "mix"):
+            raise ValueError(f"value_mix must be None, 'source' or 'mix', got {value_mix!r}")
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} heads cannot share {num_kv_heads} kv heads evenly")
         for name, v in (("chunk", chunk), ("window", window)):
@@ -50,7 +58,10 @@ class ChunkedAttention(Part):
         # the norm of queries and keys: over the whole row with a weight per column, or over each
         # head by itself with a weight of head_dim elements that all heads share
         self.norm_per_head = bool(norm_per_head)
+        if self.norm_per_head and value_mix is not None:
+            raise ValueError("values are mixed beside a norm over whole rows only")
         self.position = build_part("position", position)
+        self.value_mix, self.mix_share = value_mix, 0.0
         self.nq, self.nk = self.num_heads * self.head_dim, self.num_kv_heads * self.head_dim
         self.nv, self.no = self.num_kv_heads * self.v_head_dim, self.num_heads * self.v_head_dim
         self.w_in = self.w_o = self.q_norm = self.k_norm = self.temp = None
@@ -61,6 +72,8 @@ class ChunkedAttention(Part):
                  "v": WeightSpec((self.nv, h), MATRIX), "o": WeightSpec((h, self.no), MATRIX),
                  "q.norm": WeightSpec((self.head_dim if self.norm_per_head else self.nq,), NORM_WEIGHT),
                  "k.norm": WeightSpec((self.head_dim if self.norm_per_head else self.nk,), NORM_WEIGHT)}
+        if self.value_mix is not None:                # the source may store a number that it does not use
+            specs["vmix"] = WeightSpec((), NORM_ZERO, optional=self.value_mix == "source")
         if self.head_temperature:
             specs["temp"] = WeightSpec((self.num_heads,), NORM_WEIGHT)
         if self.head_gate:
@@ -76,6 +89,8 @@ class ChunkedAttention(Part):
         self.q_norm = as_float32(tensors["q.norm"]).contiguous()
         self.k_norm = as_float32(tensors["k.norm"]).contiguous()
         self.temp = as_float32(tensors["temp"]).contiguous() if self.head_temperature else None
+        if self.value_mix == "mix":                   # a constant of the model
+            self.mix_share = float(as_float32(tensors["vmix"]).reshape(()).item())
         if hasattr(ops, "want_row_tiles"):
             ops.want_row_tiles(self.num_heads, self.num_kv_heads)
 
@@ -88,9 +103,17 @@ class ChunkedAttention(Part):
         proj = torch.empty((t, self.w_in.shape[0]), dtype=torch.float32, device=h.device)
         ops.linear(h, self.w_in, proj)
         q = torch.empty((t, self.nq), dtype=h.dtype, device=h.device)
-        ops.qk_rownorm_rope_store(proj, self.q_norm, self.k_norm, self.eps, self.position.rotation(h.device),
-                                  step, cache, q, self.num_heads, self.num_kv_heads, self.head_dim,
-                                  self.v_head_dim, per_head=self.norm_per_head)
+        rotation = self.position.rotation(h.device)
+        if self.value_mix == "source":
+            step.scratch["value_mix"] = proj[:, self.nq + self.nk:self.nq + self.nk + self.nv]
+        if rotation.kind == "neox" or self.value_mix is not None:
+            mixed = (step.scratch["value_mix"], self.mix_share) if self.value_mix == "mix" else None
+            ops.qkv_turn_store(proj, rotation, None, step, cache, q, self.num_heads, self.num_kv_heads, self.head_dim,
+                               self.v_head_dim, row_norm=(self.q_norm, self.k_norm, self.eps), value_mix=mixed)
+        else:
+            ops.qk_rownorm_rope_store(proj, self.q_norm, self.k_norm, self.eps, rotation, step, cache, q,
+                                      self.num_heads, self.num_kv_heads, self.head_dim, self.v_head_dim,
+                                      per_head=self.norm_per_head)
         gate = proj[:, self.nq + self.nk + self.nv:] if self.head_gate else None
         out = torch.empty((t, self.no), dtype=h.dtype, device=h.device)
         ops.attention_options(q, step, cache, out, self.num_heads, self.num_kv_heads, self.head_dim,

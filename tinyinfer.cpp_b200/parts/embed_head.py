@@ -2,7 +2,8 @@
 
 Embedding: ``x[t] = float32(E[token[t]])`` without scaling (reference:
 src/inference.cu:14-24); ``scaled_sinusoid``: the row times a constant plus a sine/cosine
-wave of the token's position (``scaled``: the constant alone); ``normed``: the row under an RMSNorm with a weight of its own.  Head: ``logits = h E_out^T`` in float32, where ``E_out``
+wave of the token's position (``scaled``: the constant alone); ``normed``: the row under an RMSNorm with a weight of its own;
+``bigram``: the row plus a row of a second table that a hash of the last two tokens chooses.  Head: ``logits = h E_out^T`` in float32, where ``E_out``
 is the embedding table when the head is tied (reference: always tied,
 src/inference.cu:70-71) or a table of its own.
 """
@@ -10,7 +11,7 @@ from __future__ import annotations
 
 import torch
 
-from .base import MATRIX, NORM_WEIGHT, NORM_ZERO, Part, WeightSpec, as_float32, register_part
+from .base import MATRIX, NORM_WEIGHT, NORM_ZERO, FixedStateSpec, Part, WeightSpec, as_float32, register_part
 
 
 class Embedding(Part):
@@ -97,6 +98,36 @@ class NormedEmbedding(Embedding):
         ops.rmsnorm(rows, self.norm_weight, self.eps, out)
 
 
+class BigramEmbedding(Embedding):
+    """``x[t] = E[token[t]] + B[row]``: a second table of ``buckets + 1`` rows whose row is chosen by a
+    hash of the last two tokens, ``(token[t-1] * mul_prev + token[t] * mul_cur) mod buckets``; a
+    sequence's first token takes the last row.  The request keeps its last token."""
+
+    def __init__(self, vocab_size: int, hidden_size: int, buckets: int, mul_prev: int, mul_cur: int,
+                 tensor: str = "weight", bigram_tensor: str = "bigram"):
+        super().__init__(vocab_size, hidden_size, tensor)
+        self.buckets, self.bigram_tensor = int(buckets), str(bigram_tensor)
+        if self.buckets < 1:
+            raise ValueError(f"a hash of two tokens needs at least one bucket, got {buckets}")
+        # factors below the number of buckets give the same rows and keep the products small
+        self.mul_prev, self.mul_cur = int(mul_prev) % self.buckets, int(mul_cur) % self.buckets
+        self.bigram = None
+
+    def weight_specs(self):
+        return {self.tensor: WeightSpec((self.vocab_size, self.hidden_size), MATRIX),
+                self.bigram_tensor: WeightSpec((self.buckets + 1, self.hidden_size), MATRIX)}
+
+    def load_weights(self, tensors, ops):
+        self.table = ops.pack_linear(tensors[self.tensor])
+        self.bigram = ops.pack_linear(tensors[self.bigram_tensor])
+
+    def cache_spec(self):
+        return FixedStateSpec((1,), torch.int32)
+
+    def forward(self, ops, token_ids, out, step, cache):
+        ops.embed_bigram(self.table, self.bigram, token_ids, self.buckets, self.mul_prev, self.mul_cur, step, cache, out)
+
+
 class LMHead(Part):
     category = "head"
 
@@ -132,4 +163,5 @@ register_part("embedding", "embedding", Embedding)
 register_part("embedding", "scaled_sinusoid", SinusoidEmbedding)
 register_part("embedding", "scaled", ScaledEmbedding)
 register_part("embedding", "normed", NormedEmbedding)
+register_part("embedding", "bigram", BigramEmbedding)
 register_part("head", "lm_head", LMHead)

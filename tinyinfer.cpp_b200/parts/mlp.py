@@ -86,9 +86,12 @@ class GatedMlp(Part):
 
     ``silu``     ``silu(g) u``
     ``clamped``  ``g = min(g, limit)``, ``u = clamp(u, -limit, limit)``, ``g sigmoid(alpha g) (u + 1)``
+    ``gelu_tanh``  ``gelu(g) u`` with the tanh form of gelu
 
     The tensors are ``gate``, ``up`` and ``down``."""
     category = "ffn"
+
+    ends_in_linear = True
 
     def __init__(self, hidden_size: int, intermediate_size: int, activation: str = "clamped", limit: float = 0.0,
                  alpha: float = 1.702):

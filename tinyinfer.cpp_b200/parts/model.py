@@ -87,9 +87,23 @@ class CausalLM:
         return list(found.values())
 
     # ---- cache ---------------------------------------------------------------------------
+    @property
+    def embedding_slot(self):
+        """The cache slot of an embedding that keeps something per request, else None."""
+        return self.plan.num_cache_slots if hasattr(self.embedding, "cache_spec") else None
+
+    def cache_keys(self) -> list[tuple[int, bool]]:
+        """``(cache slot, writes)`` of every view that ``forward`` wants, each once."""
+        keys = [(e.cache_slot, e.writes_cache) for e in self.plan.schedule]
+        if self.embedding_slot is not None:
+            keys.append((self.embedding_slot, True))
+        return list(dict.fromkeys(keys))
+
     def cache_specs(self) -> list[PagedKVSpec | FixedStateSpec | None]:
         """What each cache slot of the schedule holds (from the mixer that writes it)."""
         specs: list = [None] * self.plan.num_cache_slots
+        if self.embedding_slot is not None:      # an embedding that keeps something: a slot behind the layers'
+            specs.append(self.embedding.cache_spec())
         for entry in self.plan.schedule:
             block = self.blocks[entry.layer]
             # a block that keeps something itself answers for its mixer too
@@ -107,7 +121,9 @@ class CausalLM:
         step.scratch.clear()           # what kernels derived from the step in an earlier pass is stale
         x = torch.empty((step.num_tokens, self.plan.hidden_size), dtype=torch.float32,
                         device=step.token_ids.device)
-        if getattr(self.embedding, "wants_positions", False):
+        if self.embedding_slot is not None:
+            self.embedding.forward(ops, step.token_ids, x, step, cache_views[(self.embedding_slot, True)])
+        elif getattr(self.embedding, "wants_positions", False):
             self.embedding.forward(ops, step.token_ids, x, step.positions)
         else:
             self.embedding.forward(ops, step.token_ids, x)

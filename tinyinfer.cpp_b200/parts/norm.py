@@ -1,5 +1,6 @@
 """RMSNorm: ``x * rsqrt(mean(x^2) + eps) * w``, eps inside the root, weight applied directly;
-with ``one_plus`` the stored weight lies around zero and the factor is ``1 + w``.
+with ``one_plus`` the stored weight lies around zero and the factor is ``1 + w``; with ``scalar`` the
+weight is one number for all elements; ``factor`` is a constant of the model on top of the weight.
 
 Formula as in the reference's ``rms_norm_kernel`` (src/cuda/rms_norm.cu:15-25).
 All arithmetic is float32; the result is rounded once to the output dtype.
@@ -14,20 +15,27 @@ from .base import NORM_WEIGHT, NORM_ZERO, Part, WeightSpec, as_float32, register
 class RMSNorm(Part):
     category = "norm"
 
-    def __init__(self, size: int, eps: float, tensor: str = "weight", one_plus: bool = False):
+    def __init__(self, size: int, eps: float, tensor: str = "weight", one_plus: bool = False, scalar: bool = False,
+                 factor: float = 1.0):
         self.size = int(size)
         self.eps = float(eps)
+        self.scalar, self.factor = bool(scalar), float(factor)
         self.tensor = str(tensor)            # the weight's name behind the part's prefix (may be empty)
         self.one_plus = bool(one_plus)       # the stored weight is the factor minus one
         self.weight: torch.Tensor | None = None
 
     def weight_specs(self):
-        return {self.tensor: WeightSpec((self.size,), NORM_WEIGHT)}
+        return {self.tensor: WeightSpec(() if self.scalar else (self.size,), NORM_WEIGHT)}
 
     def load_weights(self, tensors, ops):
-        self.weight = as_float32(tensors[self.tensor]).contiguous()
+        self.weight = as_float32(tensors[self.tensor])
+        if self.scalar:                              # the kernels take a weight per element
+            self.weight = self.weight.reshape(1).expand(self.size)
+        self.weight = self.weight.contiguous()
         if self.one_plus:
             self.weight = 1.0 + self.weight          # float32; the kernels multiply by it as it is
+        if self.factor != 1.0:
+            self.weight = self.factor * self.weight
 
     def forward(self, ops, x: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
         out = torch.empty((x.shape[0], self.size), dtype=out_dtype, device=x.device)
@@ -40,6 +48,15 @@ class RMSNorm(Part):
         out = torch.empty((rows.shape[0], self.size), dtype=out_dtype, device=x.device)
         ops.rmsnorm(x, self.weight, self.eps, out, rows=rows)
         return out
+
+    def forward_shifted(self, ops, x: torch.Tensor, mu: torch.Tensor, step, kept, out_dtype: torch.dtype):
+        """The normed rows ``h`` and the same rows shifted towards the token before, ``h + (h' - h) mu``
+        (``h'``: the row of the token before in its request, for a portion's first token the one that
+        ``kept`` holds, zeros at a sequence's start); ``kept`` then holds the portion's last row."""
+        h = torch.empty((x.shape[0], self.size), dtype=out_dtype, device=x.device)
+        shifted = torch.empty_like(h)
+        ops.rmsnorm_shift(x, self.weight, self.eps, mu, step, kept, h, shifted)
+        return h, shifted
 
 
 register_part("norm", "rmsnorm", RMSNorm)

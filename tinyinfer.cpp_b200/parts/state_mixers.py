@@ -24,6 +24,16 @@ maximum (the mLSTM cell of xLSTM).  ``q = Wq h * dim^-1/2``, ``k = Wk h`` (``hea
 ``o`` is brought to unit root mean square per head, the heads side by side are multiplied by a
 weight per element and by ``sigmoid(Wg h)``; then ``Wo``.
 
+``gated_linear_attention``: a decay per key channel.  ``q = Wq h * dim^-1/2``, ``k = Wk h`` (``heads x
+dim``), ``v = Wv h`` (``heads x vdim``), ``a = sigmoid(Wa2 (Wa1 h) + b)^(1/tau)`` laid out like ``k``;
+per head
+
+    S <- diag(a) S + k v^T;   o = S^T q
+
+``o`` is brought to unit root mean square per head, multiplied by a weight of ``vdim`` elements that the
+heads share and by ``silu(Wg h)``; then ``Wo``.  The inner width of the decay's two products is the
+stored tensors'; ``Wa1 h`` stays float32.
+
 All projections of a mixer run as one product.  State, gates, decays, unit norms and the
 recurrence are float32 whatever the activation dtype; the state of a request (and the
 convolution's last ``taps - 1`` inputs) lives in its state slot and starts at zero, so a prompt
@@ -150,5 +160,60 @@ class MatrixMemoryMixer(Part):
         ops.linear(out, self.w_o, residual, accumulate=True)
 
 
+class GatedLinearAttention(Part):
+    category = "mixer"
+    ends_in_linear = True
+
+    def __init__(self, hidden_size: int, num_heads: int, head_dim: int, v_head_dim: int, tau: float, norm_eps: float,
+                 decay_rank=None):
+        self.hidden_size, self.num_heads = int(hidden_size), int(num_heads)
+        self.head_dim, self.v_head_dim = int(head_dim), int(v_head_dim)
+        self.tau, self.eps = float(tau), float(norm_eps)
+        if not self.tau > 0:
+            raise ValueError(f"the decay's root must be positive, got {tau}")
+        # inner width of the decay's products: the stored tensors' own unless given (random weights need it)
+        self.decay_rank = None if decay_rank is None else int(decay_rank)
+        self.nk, self.nv = self.num_heads * self.head_dim, self.num_heads * self.v_head_dim
+        self.w_in = self.w_o = self.a2 = self.a2_bias = self.norm = None
+        self.rank = 0
+
+    def weight_specs(self):
+        h = self.hidden_size
+        return {"q": WeightSpec((self.nk, h), MATRIX), "k": WeightSpec((self.nk, h), MATRIX),
+                "v": WeightSpec((self.nv, h), MATRIX), "g": WeightSpec((self.nv, h), MATRIX),
+                "a1": WeightSpec((self.decay_rank, h), MATRIX), "a2": WeightSpec((self.nk, self.decay_rank), MATRIX),
+                "a2.b": WeightSpec((self.nk,), NORM_WEIGHT), "norm": WeightSpec((self.v_head_dim,), NORM_WEIGHT),
+                "o": WeightSpec((h, self.nv), MATRIX)}
+
+    def load_weights(self, tensors, ops):
+        # columns of the product: q, k, v, the gate, the decay's inner row
+        self.w_in = ops.pack_linear(_stack_rows([tensors[n] for n in ("q", "k", "v", "g", "a1")], self.hidden_size))
+        self.rank = tensors["a1"].shape[0]
+        self.a2 = ops.pack_linear(tensors["a2"])
+        if self.a2.shape[1] != self.rank:
+            raise ValueError(f"the decay's two matrices disagree on their inner width: {self.rank} and {self.a2.shape[1]}")
+        self.a2_bias = as_float32(tensors["a2.b"]).contiguous()
+        self.norm = as_float32(tensors["norm"]).contiguous()
+        self.w_o = ops.pack_linear(tensors["o"])
+
+    def cache_spec(self):
+        return FixedStateSpec((self.nk * self.v_head_dim,), torch.float32)
+
+    def forward(self, ops, h, residual, step, cache):
+        t, dev, nk, nv = h.shape[0], h.device, self.nk, self.nv
+        proj = torch.empty((t, self.w_in.shape[0]), dtype=torch.float32, device=dev)
+        ops.linear(h, self.w_in, proj)
+        at_g, at_a = 2 * nk + nv, 2 * nk + 2 * nv
+        decay = torch.empty((t, nk), dtype=torch.float32, device=dev)
+        ops.low_rank_decay(proj[:, at_a:at_a + self.rank], self.a2, self.a2_bias, self.tau, decay)
+        out = torch.empty((t, nv), dtype=h.dtype, device=dev)
+        ops.matrix_state("decayed_sum", proj[:, :nk], proj[:, nk:2 * nk], proj[:, 2 * nk:at_g], None, None, None, None,
+                         step, cache, out, heads=self.num_heads, kv_heads=self.num_heads, dk=self.head_dim,
+                         dv=self.v_head_dim, eps=self.eps, norm_weight=self.norm, gate=proj[:, at_g:at_a],
+                         gate_act="silu", decay=decay)
+        ops.linear(out, self.w_o, residual, accumulate=True)
+
+
+register_part("mixer", "gated_linear_attention", GatedLinearAttention)
 register_part("mixer", "gated_delta", GatedDeltaMixer)
 register_part("mixer", "matrix_memory", MatrixMemoryMixer)
