@@ -1123,6 +1123,159 @@ def nekorax_arm(args) -> int:
     return 0
 
 
+# ---- the Vametar decoder beside the Feruzen decoder at equal sizes ------------------------------
+# (width, heads, kv heads, head size, channels and blocks of the linear recurrence, taps, heads of the linear
+#  attention with their key and value size, inner width of its decay, feed-forward, blocks of [attention, linear
+#  recurrence, linear attention] layers, each with a feed-forward)
+VAMETAR_SIZES = {
+    "w1024": (1024, 16, 4, 64, 1024, 8, 4, 8, 64, 128, 16, 2816, 2),
+    "w2048": (2048, 16, 4, 128, 2048, 8, 4, 16, 128, 128, 16, 5632, 2),
+    "w4096": (4096, 32, 8, 128, 4096, 16, 4, 32, 128, 128, 16, 11008, 1),
+}
+
+
+def vametar_config(size):
+    w, h, g, d, rw, rb, taps, lh, ld, lv, rank, ff, blocks = size
+    mlp = {"kind": "dense", "ff": ff}
+    layers = [
+        {"type": "attention", "mlp": mlp, "mixer": {"heads": h, "kv_heads": g, "dim": d, "vdim": d, "scale": d ** -0.5,
+                                                    "rot": {"dims": d, "base": 500000.0}, "v_mix": True}},
+        {"type": "rglru", "mlp": mlp, "mixer": {"width": rw, "blocks": rb, "conv": taps}},
+        {"type": "gla", "mlp": mlp, "mixer": {"heads": lh, "dim": ld, "vdim": lv, "tau": 16.0, "decay_rank": rank}}]
+    return {"architecture": "Vametar", "vocab": DESIGN_VOCAB, "width": w, "norm": {"eps": 1e-6}, "residual_mult": 0.7,
+            "embedding": {"bigram": {"buckets": 8191, "mul_prev": 1009, "mul_cur": 13}}, "logit_scale": 1.0,
+            "layers": layers * blocks}
+
+
+def feruzen_beside_vametar(size):
+    """As many layers of the same width, feed-forward and heads: the delta rule, attention beside a matrix
+    memory, the delta rule again, the recurrent heads with the sizes of the linear attention's."""
+    w, h, g, d, rw, rb, taps, lh, ld, lv, rank, ff, blocks = size
+    mlp = {"kind": "dense", "ff": ff, "limit": 7.0}
+    delta = {"type": "delta", "mlp": mlp, "mixer": {"heads": lh, "kv_heads": lh, "dim": ld, "vdim": lv, "conv": taps}}
+    sides = {"type": "parallel", "mlp": mlp, "mixer": {
+        "left": {"heads": h, "kv_heads": g, "dim": d, "vdim": d, "rot": {"dims": d, "base": 500000.0}, "scale": d ** -0.5},
+        "right": {"heads": lh, "dim": ld, "vdim": lv, "gate_cap": 15.0}, "left_scale": 1.0, "right_scale": 1.0}}
+    return {"architecture": "Feruzen", "vocab": DESIGN_VOCAB, "width": w, "norm": {"eps": 1e-6, "groups": 1},
+            "canon": {"taps": taps}, "layers": [delta, sides, delta] * blocks}
+
+
+def vametar_arm(args) -> int:
+    """Prefill and decode throughput of the Vametar decoder at sizes of real layers, beside the Feruzen
+    decoder (the closest design the engine has: recurrences over a matrix state, convolutions over time,
+    attention with options and gated feed-forwards) with as many layers of the same sizes, and the time the
+    device spends in every kind of kernel call per layer, with the fraction of the roofline for the calls
+    that have one."""
+    import torch
+    from tinyinfer_b200 import Engine, StepEntry
+    pk, pk_kind = peaks()
+    prompt_len, batch, context = args.prefill_tokens, args.batch, args.context
+    warmup = max(args.warmup, 3)
+    out = {"design": "vametar", "beside": "feruzen at equal sizes", "peaks": pk_kind, "prefill_tokens": prompt_len,
+           "decode_batch": batch, "decode_context": context, "dtype": "bf16", "data": "synthetic", "sizes": {}}
+    gen = torch.Generator().manual_seed(0)
+    prompt = torch.randint(0, DESIGN_VOCAB, (prompt_len,), generator=gen).tolist()
+    hbm, tc = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12
+    # float32 multiply-adds on the CUDA cores (128 lanes an SM, the clock's maximum): what a walk over a float32 state
+    # is held against besides its bytes
+    props = torch.cuda.get_device_properties(0)
+    fp32 = props.multi_processor_count * 128 * 2.0 * getattr(props, "clock_rate", 1965000) * 1e3
+    for key, size in VAMETAR_SIZES.items():
+        if args.design_size and key != args.design_size:
+            continue
+        w, h, kvh, d, rw, rb, taps, lh, ld, lv, rank, ff, blocks = size
+        n_layers = 3 * blocks
+        res = {}
+        calls = {"vametar": ["embed_bigram", "attention_options", "qkv_turn_store", "rmsnorm_shift", "rmsnorm", "causal_conv",
+                             "conv_tail_store", "gated_recurrence", "block_products", "recurrence_rows", "low_rank_decay",
+                             "matrix_state", "glu_ffn", "gated_add", "linear"],
+                 "feruzen": ["attention_options", "qk_rownorm_rope_store", "matrix_state", "causal_conv", "conv_tail_store",
+                             "group_norm", "depth_mix", "add_scaled", "glu_ffn", "linear"]}
+        for arm, cfg in (("vametar", vametar_config(size)), ("feruzen", feruzen_beside_vametar(size))):
+            engine = Engine(config=cfg, seed=0, dtype="bfloat16", page_size=args.page_size,
+                            num_pages=-(-max(batch * context, prompt_len) // args.page_size) + batch + 2,
+                            max_requests=batch + 1, step_graphs=True)
+            pf_ms = measure_prefill(engine, prompt_len, max(1, min(args.steps, 6)), torch)
+            ms, clocks, launches = measure_decode(engine, batch, context, args.steps, warmup, torch)
+            a = {"prefill_tok_s": round(prompt_len / pf_ms * 1e3), "prefill_ms": round(pf_ms, 3),
+                 "decode_tok_s": round(batch / ms * 1e3, 1), "decode_ms_per_step": round(ms, 4),
+                 "decode_launches_per_step": launches // max(1, args.steps), "clocks": clocks}
+            engine._step_graphs = None
+            engine.ops.fuse_decode_tail = engine.ops.fuse_decode_ffn = False   # every call of its own
+            names = calls[arm]
+            for _ in range(2):        # the first eager step sizes the allocator's pool; the second is read
+                spans = timed_ops(engine, names, lambda: engine.step([StepEntry("p", prompt, [prompt_len - 1])]), torch)
+                engine.finish("p")
+            ids = fill_requests(engine, batch, context - 4, torch)
+            for _ in range(2):
+                dspans = timed_ops(engine, names, lambda: engine.step([StepEntry(r, [1 + 37 * i], [0]) for i, r in enumerate(ids)]), torch)
+            for r in ids:
+                engine.finish(r)
+            a["calls_us"] = {
+                "prompt": {n: [round(x * 1e3, 1) for x in v[:12]] for n, v in spans.items() if not n.startswith("_") and n != "linear"},
+                "decode": {n: [round(x * 1e3, 1) for x in v[:12]] for n, v in dspans.items() if not n.startswith("_") and n != "linear"}}
+            a["per_layer_us"] = {
+                "prompt": {n: round(sum(v) / n_layers * 1e3, 1) for n, v in spans.items() if not n.startswith("_")},
+                "decode": {n: round(sum(v) / n_layers * 1e3, 1) for n, v in dspans.items() if not n.startswith("_")}}
+            seen_all = prompt_len * (prompt_len + 1) / 2
+
+            def frac(amount, ms_, peak):
+                return round(amount / (ms_ * 1e-3) / peak, 4)
+
+            def product(sp, shape):
+                """The first closing product (one that adds to the residual) with a weight of this shape."""
+                return next(ms_ for ms_, (s, acc) in zip(sp["linear"], sp["_linear_kinds"]) if s == shape and acc)
+
+            att, datt = spans["attention_options"], dspans["attention_options"]
+            lin_rows = prompt_len * ((2 * lh * ld + 2 * lh * lv) * 4 + lh * lv * 2.0)
+            cols = (h + 2 * kvh) * d
+            a["roofline_frac"] = {
+                "prompt_attention": frac(4.0 * h * d * seen_all, att[0], tc),
+                "decode_attention": frac(batch * kvh * context * 2 * d * 2.0, datt[0], hbm),
+                "prompt_ffn": frac(2.0 * prompt_len * 3 * w * ff, spans["glu_ffn"][0], tc),
+                "decode_ffn": frac(2.0 * 3 * w * ff, dspans["glu_ffn"][0], hbm),
+                # the product behind the attention, with what it does to the residual
+                "prompt_closing_product": frac(2.0 * prompt_len * w * h * d, product(spans, (w, h * d)), tc),
+                "decode_closing_product": frac(2.0 * w * h * d, product(dspans, (w, h * d)), hbm)}
+            if arm == "vametar":
+                st, dst = spans["matrix_state"], dspans["matrix_state"]
+                walk = (rw * (4 * 4 + 2.0)) * prompt_len
+                a["roofline_frac"].update({
+                    "prompt_linear_attention_fp32": frac(prompt_len * lh * ld * lv * 5.0, st[0], fp32),
+                    "prompt_linear_attention_bytes": frac(lin_rows + prompt_len * lh * ld * 4.0, st[0], hbm),
+                    "decode_linear_attention_state_bytes": frac(batch * lh * ld * lv * 8.0, dst[0], hbm),
+                    "prompt_key_decays_bytes": frac(prompt_len * lh * ld * 4.0, spans["low_rank_decay"][0], hbm),
+                    "prompt_recurrence_products": frac(2.0 * prompt_len * 2 * rw * (rw // rb), spans["block_products"][0], tc),
+                    "prompt_recurrence_bytes": frac(walk, spans["recurrence_rows"][0], hbm),
+                    "decode_recurrence_bytes": frac(4.0 * rw * (rw // rb) + batch * rw * 18.0, dspans["gated_recurrence"][0], hbm),
+                    "prompt_convolution": frac(prompt_len * rw * 8.0, spans["causal_conv"][0], hbm),
+                    "prompt_norm_and_shift": frac(prompt_len * w * (4 + 2 + 2.0), spans["rmsnorm_shift"][0], hbm),
+                    "prompt_norm": frac(prompt_len * w * (4 + 2.0), spans["rmsnorm"][0], hbm),
+                    "prompt_norm_turn_and_store": frac(prompt_len * cols * (4 + 2.0), spans["qkv_turn_store"][0], hbm)})
+            else:
+                # a block's layers: delta rule, attention beside the memory, delta rule
+                st, dst = spans["matrix_state"], dspans["matrix_state"]
+                mem_rows = lin_rows + prompt_len * 2 * lh * 4.0
+                a["roofline_frac"].update({
+                    "prompt_delta_rule_fp32": frac(prompt_len * lh * ld * lv * 7.0, st[0], fp32),
+                    "prompt_matrix_memory_fp32": frac(prompt_len * lh * ld * (lv + 1) * 5.0, st[1], fp32),
+                    "prompt_delta_rule_bytes": frac(mem_rows, st[0], hbm),
+                    "prompt_matrix_memory_bytes": frac(mem_rows, st[1], hbm),
+                    "decode_delta_rule_state_bytes": frac(batch * lh * ld * lv * 8.0, dst[0], hbm),
+                    "decode_matrix_memory_state_bytes": frac(batch * lh * ld * (lv + 1) * 8.0, dst[1], hbm),
+                    # the first convolution of a layer runs over the width, the second over q, k, v
+                    "prompt_convolution": frac(prompt_len * (2 * lh * ld + lh * lv) * 8.0, spans["causal_conv"][1], hbm),
+                    "prompt_norm_added": frac(prompt_len * w * (4 + 4 + 4.0), spans["group_norm"][0], hbm),
+                    "prompt_norm_turn_and_store": frac(prompt_len * cols * (4 + 2.0), spans["qk_rownorm_rope_store"][0], hbm)})
+            res[arm] = a
+            del engine
+            torch.cuda.empty_cache()
+        out["sizes"][key] = {"width": w, "heads": h, "kv_heads": kvh, "head_dim": d, "recurrence": [rw, rb], "taps": taps,
+                             "linear_attention": [lh, ld, lv], "decay_rank": rank, "ff": ff, "layers": n_layers, **res}
+    print(json.dumps(out))
+    return 0
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1142,9 +1295,9 @@ def main() -> int:
                     help="with --only mixed: the number of decoding requests beside the 512-token portion")
     ap.add_argument("--attention-in-turn", action="store_true",
                     help="with --only mixed: flash-decoding behind the prompt attention kernel, not beside it")
-    ap.add_argument("--design", choices=["kagorax", "ruvuvik", "feruzen", "nekorax"], default=None,
-                    help="set this decoder beside the closest one the engine has (Qwen3; for feruzen and nekorax: Ruvuvik) at equal sizes instead of the default run")
-    ap.add_argument("--design-size", choices=sorted(set(DESIGN_SIZES) | set(RUVUVIK_SIZES) | set(FERUZEN_SIZES) | set(NEKORAX_SIZES)), default=None,
+    ap.add_argument("--design", choices=["kagorax", "ruvuvik", "feruzen", "nekorax", "vametar"], default=None,
+                    help="set this decoder beside the closest one the engine has (Qwen3; for feruzen and nekorax: Ruvuvik; for vametar: Feruzen) at equal sizes instead of the default run")
+    ap.add_argument("--design-size", choices=sorted(set(DESIGN_SIZES) | set(RUVUVIK_SIZES) | set(FERUZEN_SIZES) | set(NEKORAX_SIZES) | set(VAMETAR_SIZES)), default=None,
                     help="one of the sizes only")
     ap.add_argument("--only", choices=["decode", "prefill", "chains", "mixed"], default=None,
                     help="run one part only and print a short line (for profiling small cases)")
@@ -1162,6 +1315,8 @@ def main() -> int:
         return feruzen_arm(args)
     if args.design == "nekorax":
         return nekorax_arm(args)
+    if args.design == "vametar":
+        return vametar_arm(args)
     if args.design:
         return design_arm(args)
 

@@ -392,7 +392,18 @@ class StateOps:
                 state.slots.data_ptr(), step.num_requests, n, st.data_ptr(), st.stride(0), out.data_ptr(),
                 _CODE[out.dtype], self._stream()))
             return
+        z, row_stride, block_stride = self.block_products(u, gates, fast)
+        self.recurrence_rows(u, z, row_stride, block_stride, gate_bias, per, log_decay, y, y_bias, step, state, out)
+
+    def block_products(self, u, gates, fast):
+        """``Wr[b] u_b`` and ``Wi[b] u_b`` for every row of the float32 ``u``, with float32 sums.  Returns the
+        float32 rows, the stride from a token to the next and the stride from a block to the next; a
+        block's ``per`` columns of the first product lie in front of those of the second.  ``fast``: many
+        rows may take the tensor cores."""
+        t, n = u.shape
+        blocks, per = gates.blocks, gates.per
         if fast and t > 64 and per % 8 == 0 and gates.rows.dtype == torch.bfloat16:
+            lib = self.channels_lib
             padded = -(-t // 128) * 128
             cut = torch.empty((blocks, padded, 3 * per), dtype=torch.bfloat16, device=u.device)
             self._ch(lib.ti_split_rows(u.data_ptr(), u.stride(0), t, n, per, padded, cut.data_ptr(), self._stream()))
@@ -402,16 +413,20 @@ class StateOps:
                 cut.data_ptr(), gates.thrice.data_ptr(), z.data_ptr(), None, blocks * padded, 2 * per, 3 * per, 3 * per,
                 3 * per, 2 * per, 0, 0, blocks, group_of_tile.data_ptr(), tiles.data_ptr(), self.status.data_ptr(),
                 self._stream()), self.bf16)
-            row_stride, block_stride = 2 * per, padded * 2 * per
+            return z, 2 * per, padded * 2 * per
+        z = torch.empty((t, blocks, 2 * per), dtype=torch.float32, device=u.device)
+        if per <= 768:
+            self.head_project(u.unflatten(1, (blocks, per)), gates.cols, z)
         else:
-            z = torch.empty((t, blocks, 2 * per), dtype=torch.float32, device=u.device)
-            if per <= 768:
-                self.head_project(u.view(t, blocks, per), gates.cols, z)
-            else:
-                for b in range(blocks):
-                    self.linear(u[:, b * per:(b + 1) * per], gates.rows[b], z[:, b])
-            row_stride, block_stride = 2 * n, 2 * per
-        self._ch(lib.ti_gated_recurrence(
+            for b in range(blocks):
+                self.linear(u[:, b * per:(b + 1) * per], gates.rows[b], z[:, b])
+        return z, 2 * n, 2 * per
+
+    def recurrence_rows(self, u, z, row_stride, block_stride, gate_bias, per, log_decay, y, y_bias, step, state, out):
+        """The walk of ``gated_recurrence`` behind its products (``z`` and its strides: ``block_products``)."""
+        t, n = out.shape
+        st = state.state
+        self._ch(self.channels_lib.ti_gated_recurrence(
             u.data_ptr(), u.stride(0), z.data_ptr(), row_stride, block_stride, y.data_ptr(), y.stride(0),
             gate_bias.data_ptr(), per, log_decay.data_ptr(), y_bias.data_ptr(), step.cu_q.data_ptr(),
             state.slots.data_ptr(), step.num_requests, n, st.data_ptr(), st.stride(0), out.data_ptr(), _CODE[out.dtype],
