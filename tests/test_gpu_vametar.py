@@ -141,7 +141,7 @@ def test_norm_and_token_shift_over_portions(ops, width, dtype):
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("sizes", [(1, 48, 32), (5, 40, 24), (8, 1024, 256), (3, 4096, 512), (17, 130, 96), (64, 256, 4096), (90, 256, 128),
                                    (70, 52, 40), (513, 1024, 320), (300, 300, 64), (2000, 512, 192), (129, 6144, 4096),
-                                   (40, 5120, 4096)])
+                                   (40, 5120, 4096), (1100, 2560, 64)])
 def test_products_that_pass_a_gate(ops, sizes, dtype):
     """``x += scale sigmoid(gate + bias) (a w^T)`` for the sizes that every form of the product takes."""
     from tinyinfer_b200.parts.base import GatedSum
@@ -162,6 +162,43 @@ def test_products_that_pass_a_gate(ops, sizes, dtype):
     d = x.to(DEV)
     ops.gated_add(y.float().to(DEV), GatedSum(d, gate.to(DEV)[:, 4:4 + n], bias.to(DEV), -0.7))
     _close(d - x.to(DEV), add, torch.float32, "added")
+
+
+@pytest.mark.parametrize("sizes", [(1, 64, 48, 40), (8, 1024, 3072, 1024), (3, 96, 64, 2080), (16, 2048, 48, 2048), (33, 128, 512, 256),
+                                   (64, 40, 40, 64), (8, 72, 16, 96)])
+def test_two_products_of_few_rows_in_one_launch(ops, sizes):
+    """A product that waits for the next one gives the same bits as by itself, beside a plain product and
+    beside one whose epilogue is a gated activation; what cannot share a launch is launched by itself."""
+    t, n1, n2, k = sizes
+    g = torch.Generator().manual_seed(n1)
+    rand = lambda *s: (torch.randn(s, generator=g) / s[-1] ** 0.5).to(torch.bfloat16).to(DEV)
+    a1, a2, w1, w2 = rand(t, k), rand(t, k), rand(n1, k), rand(n2, k)
+    gate_up, down = ops.pack_gate_up(rand(n2, k), rand(n2, k)), rand(k, n2)
+    empty = lambda n: torch.full((t, n), float("nan"), dtype=torch.float32, device=DEV)
+
+    def both(pair):
+        ops.pair_few_rows = pair
+        before, outs = ops.launches, [empty(n1), empty(n2), empty(n1), torch.zeros((t, k), device=DEV), empty(n1), empty(n2)]
+        ops.linear(a1, w1, outs[0], may_pair=True)
+        ops.linear(a2, w2, outs[1])
+        ops.linear(a1, w1, outs[2], may_pair=True)
+        ops.glu_ffn(a2, gate_up, down, outs[3], "gelu_tanh", 0.0, 0.0)
+        count = ops.launches - before
+        ops.linear(a1, w1, outs[4], may_pair=True)
+        ops.linear(a1[:, :32].contiguous(), w2[:, :32].contiguous(), outs[5])          # another k
+        ops.linear(a1, w1, outs[0], may_pair=True)
+        ops.flush()
+        return outs, count
+
+    try:
+        (apart, more), (together, fewer) = both(False), both(True)
+    finally:
+        ops.pair_few_rows = True
+    assert fewer < more or k % 32 != 0
+    for x, y in zip(apart, together):
+        assert torch.equal(x, y)
+    want = a2.double() @ w2.double().T
+    _close(together[1], want.cpu(), torch.bfloat16, "second product")
 
 
 @pytest.mark.parametrize("taps", [1, 2, 4, 7])

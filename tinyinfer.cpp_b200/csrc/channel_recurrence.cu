@@ -5,10 +5,9 @@
 //  * gated_recurrence: per channel, over a request's tokens in order,
 //        a = exp(L sigmoid(zr + br));   S <- a S + sqrt(1 - a^2) sigmoid(zi + bi) u;   out = S gelu(y + by)
 //    with L <= 0 a constant of the channel and S in the request's state slot.  One block walks a request's
-//    tokens for 32 channels (a lane each): seven warps turn a tile's inputs into (a, b) pairs and finished
+//    tokens for 8, 16 or 32 channels: fifteen warps turn a tile's inputs into (a, b) pairs and finished
 //    states into output rows, one warp does nothing but S <- a S + b.  While it walks tile i, the others
-//    prepare tile i + 1, write out tile i - 1 and have the loads of the tiles behind on their way, so a
-//    portion takes about as long as its bytes need.  Every channel's chain is one multiply-add per token in
+//    prepare tile i + 1, write out tile i - 1 and have the loads of the tiles behind on their way.  Every channel's chain is one multiply-add per token in
 //    order, so a row's bits depend neither on the batch nor on how a prompt was cut.
 //  * gated_recurrence_single: the same for steps in which every request brings one token, with the block-
 //    diagonal products z = W u in front.  A block takes 16 channels of a part: its warps read the 32 rows of W
@@ -16,7 +15,6 @@
 //  * split_rows: a float32 row as three bfloat16 rows that add up to it (24 of its 24 bits), laid out so that
 //    one grouped tensor-core product with a weight that repeats itself three times along k gives float32 sums.
 #include "common.cuh"
-#include "glu.cuh"
 
 namespace {
 
@@ -69,12 +67,18 @@ low_rank_decay_kernel(const float* low, int low_stride, int rank, const TW* __re
 // ---- the recurrence ---------------------------------------------------------------------------------
 struct Channel { float br, bi, log_decay, by; };
 
-__device__ __forceinline__ float sigmoidf_(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float sigmoidf_(float z) { return __fdividef(1.0f, 1.0f + expf(-z)); }
 
-// (a, b) of S <- a S + b for one token
+// (a, b) of S <- a S + b for one token: a = e^l, b = sqrt(1 - a^2) i u, both from e^l - 1 (1 - a^2 = -e (2 + e) keeps its
+// digits where a is near 1)
 __device__ __forceinline__ float2 gate_pair(const Channel& p, float zr, float zi, float u) {
-    const float log_a = p.log_decay * sigmoidf_(zr + p.br);
-    return make_float2(expf(log_a), sqrtf(-expm1f(2.0f * log_a)) * sigmoidf_(zi + p.bi) * u);
+    const float e = expm1f(p.log_decay * sigmoidf_(zr + p.br));
+    return make_float2(1.0f + e, sqrtf(-e * (2.0f + e)) * sigmoidf_(zi + p.bi) * u);
+}
+
+// gelu(z), the tanh form: 1/2 (1 + tanh x) = sigmoid(2 x)
+__device__ __forceinline__ float gelu_gate(float z) {
+    return z * sigmoidf_(1.5957691216057308f * fmaf(0.044715f * z * z, z, z));
 }
 
 struct RecurrenceArgs {
@@ -92,32 +96,42 @@ __device__ __forceinline__ Channel channel_of(const RecurrenceArgs& p, int c) {
     return {p.gate_bias[c], p.gate_bias[p.width + c], p.log_decay[c], p.y_bias[c]};
 }
 
-constexpr int GR_WARPS = 8, GR_ROWS = 8, GR_TILE = (GR_WARPS - 1) * GR_ROWS;      // 56 tokens a tile, eight a warp
+// CH channels a block; a warp's lanes are CH channels of 32 / CH neighbouring tokens
+constexpr int GR_WARPS = 16, GR_ROWS = 4, GR_BATCH = 12;
+template <int CH> struct RecurrenceTile {
+    static constexpr int tokens_at_once = 32 / CH;
+    static constexpr int tokens_warp = GR_ROWS * tokens_at_once;
+    static constexpr int tokens = (GR_WARPS - 1) * tokens_warp;             // 60 x 32 / CH
+    static_assert(tokens % GR_BATCH == 0, "whole batches of the walk");
+};
 
-template <typename TO>
+template <typename TO, int CH>
 __global__ void __launch_bounds__(GR_WARPS * 32)
 gated_recurrence_kernel(const RecurrenceArgs p, TO* __restrict__ out) {
-    __shared__ float2 ab[2][GR_TILE][32];
-    __shared__ float ss[2][GR_TILE][32];
+    using Tile = RecurrenceTile<CH>;
+    constexpr int TT = Tile::tokens;
+    __shared__ float2 ab[2][TT][CH];
+    __shared__ float ss[2][TT][CH];
     const int req = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t0 = p.cu_q[req], t1 = p.cu_q[req + 1];
     if (t0 >= t1) return;
-    const int c = blockIdx.y * 32 + lane;
+    const int j = lane % CH, c = blockIdx.y * CH + j;
     const bool live = c < p.width;
     const int cc = live ? c : p.width - 1;                // lanes past the width read the last channel and store nothing
     const Channel ch = channel_of(p, cc);
     const float* gp = p.gates + (size_t)(cc / p.per) * p.gates_block + cc % p.per;
     const float* up = p.u + cc;
     const float* yp = p.y + cc;
-    const int tiles = (t1 - t0 + GR_TILE - 1) / GR_TILE;
-    const int row0 = (warp - 1) * GR_ROWS;                // this warp's rows of a tile (warps 1 to 7)
+    const int tiles = (t1 - t0 + TT - 1) / TT;
+    const int row0 = (warp - 1) * Tile::tokens_warp + lane / CH;            // this lane's first token of a tile (warps 1 to 15)
     float* slot = p.state + (size_t)p.slots[req] * p.state_stride + cc;
 
     float zr[GR_ROWS], zi[GR_ROWS], u[GR_ROWS], y[GR_ROWS], y_next[GR_ROWS];
+    auto row = [&](int i) { return row0 + i * Tile::tokens_at_once; };
     auto fetch = [&](int tile) {                          // the inputs of a tile's (a, b), on their way
 #pragma unroll
         for (int i = 0; i < GR_ROWS; ++i) {
-            const int t = t0 + tile * GR_TILE + row0 + i;
+            const int t = t0 + tile * TT + row(i);
             const bool in = t < t1;
             const float* g = gp + (size_t)(in ? t : t0) * p.gates_stride;
             zr[i] = g[0];
@@ -128,20 +142,20 @@ gated_recurrence_kernel(const RecurrenceArgs p, TO* __restrict__ out) {
     auto fetch_y = [&](int tile, float (&dst)[GR_ROWS]) {
 #pragma unroll
         for (int i = 0; i < GR_ROWS; ++i) {
-            const int t = t0 + tile * GR_TILE + row0 + i;
+            const int t = t0 + tile * TT + row(i);
             dst[i] = yp[(size_t)(t < t1 ? t : t0) * p.y_stride];
         }
     };
     auto prepare = [&](int buf) {
 #pragma unroll
-        for (int i = 0; i < GR_ROWS; ++i) ab[buf][row0 + i][lane] = gate_pair(ch, zr[i], zi[i], u[i]);
+        for (int i = 0; i < GR_ROWS; ++i) ab[buf][row(i)][j] = gate_pair(ch, zr[i], zi[i], u[i]);
     };
     auto finish = [&](int tile) {
 #pragma unroll
         for (int i = 0; i < GR_ROWS; ++i) {
-            const int t = t0 + tile * GR_TILE + row0 + i;
+            const int t = t0 + tile * TT + row(i);
             if (t < t1 && live)
-                out[(size_t)t * p.width + c] = from_f32<TO>(ss[tile & 1][row0 + i][lane] * gelu_tanh(y[i] + ch.by));
+                out[(size_t)t * p.width + c] = from_f32<TO>(ss[tile & 1][row(i)][j] * gelu_gate(y[i] + ch.by));
         }
     };
     float S = 0.0f;
@@ -156,21 +170,25 @@ gated_recurrence_kernel(const RecurrenceArgs p, TO* __restrict__ out) {
     __syncthreads();
     for (int tile = 0; tile < tiles; ++tile) {
         if (warp == 0) {
-            const int nt = min(GR_TILE, t1 - t0 - tile * GR_TILE);
-            const float2 (*from)[32] = ab[tile & 1];
-            float (*to)[32] = ss[tile & 1];
-            if (nt == GR_TILE) {
-#pragma unroll 14
-                for (int i = 0; i < GR_TILE; ++i) {
-                    const float2 v = from[i][lane];
-                    S = fmaf(v.x, S, v.y);
-                    to[i][lane] = S;
+            if (lane < CH) {
+                const int nt = min(TT, t1 - t0 - tile * TT);
+                const float2 (*from)[CH] = ab[tile & 1];
+                float (*to)[CH] = ss[tile & 1];
+                int i = 0;
+                for (; i + GR_BATCH <= nt; i += GR_BATCH) {        // a batch's pairs first: the chain then waits for itself alone
+                    float2 v[GR_BATCH];
+#pragma unroll
+                    for (int b = 0; b < GR_BATCH; ++b) v[b] = from[i + b][j];
+#pragma unroll
+                    for (int b = 0; b < GR_BATCH; ++b) {
+                        S = fmaf(v[b].x, S, v[b].y);
+                        to[i + b][j] = S;
+                    }
                 }
-            } else {
-                for (int i = 0; i < nt; ++i) {
-                    const float2 v = from[i][lane];
+                for (; i < nt; ++i) {
+                    const float2 v = from[i][j];
                     S = fmaf(v.x, S, v.y);
-                    to[i][lane] = S;
+                    to[i][j] = S;
                 }
             }
         } else {
@@ -186,7 +204,7 @@ gated_recurrence_kernel(const RecurrenceArgs p, TO* __restrict__ out) {
         __syncthreads();
     }
     if (warp == 0) {
-        if (live) *slot = S;
+        if (live && lane < CH) *slot = S;
     } else {
         finish(tiles - 1);
     }
@@ -282,7 +300,7 @@ gated_recurrence_single_kernel(const RecurrenceArgs p, const TW* __restrict__ w,
         const float2 v = gate_pair(ch, z[i][r], z[GS_CHANNELS + i][r], us[(size_t)r * p.per + c0 + i]);
         const float S = fmaf(v.x, *slot, v.y);
         *slot = S;
-        out[(size_t)t * p.width + c] = from_f32<TO>(S * gelu_tanh(p.y[(size_t)t * p.y_stride + c] + ch.by));
+        out[(size_t)t * p.width + c] = from_f32<TO>(S * gelu_gate(p.y[(size_t)t * p.y_stride + c] + ch.by));
     }
 }
 
@@ -350,12 +368,25 @@ extern "C" int ti_gated_recurrence(const float* u, int u_stride, const float* ga
     TI_REQUIRE(per >= 1 && width % per == 0, "gated_recurrence: %d channels in parts of %d", width, per);
     const RecurrenceArgs a = recurrence_args(u, u_stride, gates, gates_stride, gates_block, y, y_stride, gate_bias, per,
                                              log_decay, y_bias, cu_q, slots, width, state, state_stride);
-    const dim3 grid(requests, (width + 31) / 32);
+    int device = 0, sms = 0;
+    cudaGetDevice(&device);
+    cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, device);
+    // few blocks: fewer channels each, so that more SMs share the gates' exponentials (the bits do not depend on it)
+    int ch = 32;
+    while (ch > 8 && (long long)requests * ((width + ch / 2 - 1) / (ch / 2)) <= 2LL * sms) ch /= 2;
+    const dim3 grid(requests, (width + ch - 1) / ch);
     TI_REQUIRE(grid.y <= 65535, "gated_recurrence: %d channels", width);
+    TI_REQUIRE(out_dtype == TI_BF16 || out_dtype == TI_F32, "gated_recurrence: output dtype code %d", out_dtype);
     cudaStream_t s = (cudaStream_t)stream;
-    if (out_dtype == TI_BF16) gated_recurrence_kernel<bf16><<<grid, GR_WARPS * 32, 0, s>>>(a, (bf16*)out);
-    else if (out_dtype == TI_F32) gated_recurrence_kernel<float><<<grid, GR_WARPS * 32, 0, s>>>(a, (float*)out);
-    else return ti_fail("gated_recurrence: output dtype code %d", out_dtype);
+#define CALL(CH)                                                                                                     \
+    do {                                                                                                             \
+        if (out_dtype == TI_BF16) gated_recurrence_kernel<bf16, CH><<<grid, GR_WARPS * 32, 0, s>>>(a, (bf16*)out);     \
+        else gated_recurrence_kernel<float, CH><<<grid, GR_WARPS * 32, 0, s>>>(a, (float*)out);                        \
+    } while (0)
+    if (ch == 32) CALL(32);
+    else if (ch == 16) CALL(16);
+    else CALL(8);
+#undef CALL
     return ti_check_launch("gated_recurrence");
 }
 

@@ -10,7 +10,8 @@
 // block are added in a fixed order in shared memory, so an output does not depend on M, on the
 // other rows or on the launch.
 //
-// Epilogues: store, accumulate into C (the residual stream), or SwiGLU: W holds, in every strip,
+// Epilogues: store, accumulate into C (the residual stream; optionally through a gate, C += scale
+// sigmoid(gate + bias) * sum), or SwiGLU: W holds, in every strip,
 // 8 gate rows followed by their 8 up rows, and out[m, j] = silu(gate_j) * up_j in bfloat16.
 #include "common.cuh"
 #include "glu.cuh"
@@ -38,6 +39,11 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], unsigned a0, unsigned a1
                  : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
 
+// A second product over the same number of rows and the same k in the same launch: the blocks from `first_block` on
+// (0: there is none) store its strips.  Two products of a decode step that depend on nothing of each other (a
+// sublayer's first product and its gate) then wait for the kernel before them once.
+struct SecondProduct { const bf16* a; const bf16* w; float* c; int n, lda, ldw, ldc; unsigned first_block; };
+
 // ROWS = 16: a block owns 16 rows of W.  ROWS = 8: it owns 8 (the upper half of the MMA's A
 // operand is zero), which doubles the number of blocks for narrow outputs.
 constexpr int SHORT_K = WARPS * CHUNK * 4;     // what four chunks per warp cover: 1,024
@@ -49,13 +55,20 @@ template <int NT, int ROWS, int BATCH, bool STORE_ONLY = false>
 __global__ void __launch_bounds__(WARPS * 32, BATCH == 4 && NT == 1 ? 3 : 2)
 gemm_skinny_kernel(const bf16* a, const bf16* __restrict__ w, float* __restrict__ c,
                    bf16* __restrict__ out_act, int m, int n, int k, int lda, int ldw, int ldc,
-                   int ld_act, int mode, int glu_kind, float act_p, float act_q) {
+                   int ld_act, int mode, int glu_kind, float act_p, float act_q, const AddGate add,
+                   const SecondProduct second) {
     constexpr int MP = NT * 8;                                  // padded token count
     __shared__ float part[WARPS][ROWS][MP + 1];
     if (STORE_ONLY) mode = MODE_STORE;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int g = lane >> 2, tq = lane & 3;
-    const int n0 = blockIdx.x * ROWS;
+    int n0 = blockIdx.x * ROWS;
+    if (second.first_block > 0 && blockIdx.x >= second.first_block) {      // the blocks of the second product
+        n0 = (blockIdx.x - second.first_block) * ROWS;
+        a = second.a; w = second.w; c = second.c;
+        n = second.n; lda = second.lda; ldw = second.ldw; ldc = second.ldc;
+        mode = MODE_STORE;
+    }
     // rows past N are read from the last row and never stored
     const bf16* w_lo = w + (size_t)min(n0 + g, n - 1) * ldw + tq * 8;
     const bf16* w_hi = w + (size_t)min(n0 + g + 8, n - 1) * ldw + tq * 8;
@@ -125,6 +138,7 @@ gemm_skinny_kernel(const bf16* a, const bf16* __restrict__ w, float* __restrict_
     // exchanged (read one by one between the stores below, each would wait a round trip to L2).
     constexpr int OUT_STEP = WARPS * 32 / ROWS;                 // tokens a pass of the block covers
     float old_c[8 * NT / OUT_STEP > 0 ? 8 * NT / OUT_STEP : 1];
+    float gate_c[8 * NT / OUT_STEP > 0 ? 8 * NT / OUT_STEP : 1];
     if (mode == MODE_ACCUMULATE) {
         if (chunks <= warp) pdl_wait();
         const int i = threadIdx.x % ROWS;
@@ -132,6 +146,7 @@ gemm_skinny_kernel(const bf16* a, const bf16* __restrict__ w, float* __restrict_
         for (int it = 0; it < (int)(sizeof(old_c) / sizeof(float)); ++it) {
             const int tok = threadIdx.x / ROWS + it * OUT_STEP;
             old_c[it] = tok < m && n0 + i < n ? __ldcg(c + (size_t)tok * ldc + n0 + i) : 0.0f;
+            gate_c[it] = add.gate && tok < m && n0 + i < n ? __ldcg(add.gate + (size_t)tok * add.ld + n0 + i) + add.bias[n0 + i] : 0.0f;
         }
     }
     // acc[j]: [0],[1] = W row g, tokens 8j + 2tq (+1); [2],[3] = W row g + 8
@@ -174,7 +189,7 @@ gemm_skinny_kernel(const bf16* a, const bf16* __restrict__ w, float* __restrict_
                 const float y = sum > 0.0f ? fmaf(act_p * sum, sum, 0.5f * sum) : fmaf(act_q, expm1f(sum) - sum, 0.5f * sum);
                 if (n0 + i < n) out_act[(size_t)tok * ld_act + n0 + i] = __float2bfloat16_rn(y);
             } else if (n0 + i < n) {
-                c[(size_t)tok * ldc + n0 + i] = mode == MODE_ACCUMULATE ? old_c[it] + sum : sum;
+                c[(size_t)tok * ldc + n0 + i] = mode == MODE_ACCUMULATE ? add_through(add, old_c[it], sum, gate_c[it], 0.0f) : sum;
             }
         }
     }
@@ -189,7 +204,9 @@ extern "C" int ti_gemm_skinny_supported(int m, int n, int k, int lda, int ldw) {
 // mode 0: c = a w^T; 1: c += a w^T; 2: out_act[m, n/2] = swiglu over strips of 8 gate + 8 up rows;
 // 3: out_act[m, n] = xielu(a w^T) with the activation's two factors.
 static int skinny(const void* a, const void* w, float* c, void* out_act, int m, int n, int k, int lda, int ldw,
-                  int ldc, int ld_act, int mode, int glu_kind, float act_p, float act_q, void* stream) {
+                  int ldc, int ld_act, int mode, int glu_kind, float act_p, float act_q, void* stream,
+                  AddGate add = AddGate{nullptr, 0, nullptr, 0.0f},
+                  SecondProduct second = SecondProduct{nullptr, nullptr, nullptr, 0, 0, 0, 0, 0}) {
     if (m == 0 || n == 0) return 0;
     TI_REQUIRE(ti_gemm_skinny_supported(m, n, k, lda, ldw),
                "gemm_skinny: M=%d (1..64), K=%d (multiple of 32) or row strides %d, %d (multiples of 8) "
@@ -199,24 +216,30 @@ static int skinny(const void* a, const void* w, float* c, void* out_act, int m, 
     TI_REQUIRE(mode != MODE_SWIGLU || n % 16 == 0, "gemm_skinny: SwiGLU needs N %% 16 == 0, got %d", n);
     cudaStream_t s = (cudaStream_t)stream;
     // narrow outputs get blocks of 8 rows, so that at least about 128 blocks share the reading
-    const bool narrow = mode != MODE_SWIGLU && (n + STRIP - 1) / STRIP < 128;
+    const bool narrow = mode != MODE_SWIGLU && (n + STRIP - 1) / STRIP + (second.n + STRIP - 1) / STRIP < 128;
+    const int rows = narrow ? 8 : STRIP;
+    unsigned blocks = (unsigned)((n + rows - 1) / rows);
+    if (second.n > 0) {
+        second.first_block = blocks;
+        blocks += (unsigned)((second.n + rows - 1) / rows);
+    }
 #define LAUNCH(NT)                                                                                  \
     if (narrow)                                                                                     \
-        ti_launch_pdl(gemm_skinny_kernel<NT, 8, 8>, (unsigned)((n + 7) / 8), WARPS * 32, 0, s,      \
+        ti_launch_pdl(gemm_skinny_kernel<NT, 8, 8>, blocks, WARPS * 32, 0, s,      \
                       (const bf16*)a, (const bf16*)w, c, (bf16*)out_act, m, n, k, lda, ldw, ldc,    \
-                      ld_act, mode, glu_kind, act_p, act_q);                                                                \
+                      ld_act, mode, glu_kind, act_p, act_q, add, second);                                                                \
     else if (k <= SHORT_K && mode == MODE_STORE && NT <= 2)                                         \
-        ti_launch_pdl((gemm_skinny_kernel<NT <= 2 ? NT : 1, 16, 4, true>), (unsigned)((n + STRIP - 1) / STRIP), \
+        ti_launch_pdl((gemm_skinny_kernel<NT <= 2 ? NT : 1, 16, 4, true>), blocks, \
                       WARPS * 32, 0, s, (const bf16*)a, (const bf16*)w, c, (bf16*)out_act, m, n, k, \
-                      lda, ldw, ldc, ld_act, mode, glu_kind, act_p, act_q);                                   \
+                      lda, ldw, ldc, ld_act, mode, glu_kind, act_p, act_q, add, second);                                   \
     else if (k <= SHORT_K)                                                                          \
-        ti_launch_pdl(gemm_skinny_kernel<NT, 16, 4>, (unsigned)((n + STRIP - 1) / STRIP),           \
+        ti_launch_pdl(gemm_skinny_kernel<NT, 16, 4>, blocks,                                        \
                       WARPS * 32, 0, s, (const bf16*)a, (const bf16*)w, c, (bf16*)out_act, m, n, k, \
-                      lda, ldw, ldc, ld_act, mode, glu_kind, act_p, act_q);                                   \
+                      lda, ldw, ldc, ld_act, mode, glu_kind, act_p, act_q, add, second);                                   \
     else                                                                                            \
-        ti_launch_pdl(gemm_skinny_kernel<NT, 16, 8>, (unsigned)((n + STRIP - 1) / STRIP),           \
+        ti_launch_pdl(gemm_skinny_kernel<NT, 16, 8>, blocks,                                        \
                       WARPS * 32, 0, s, (const bf16*)a, (const bf16*)w, c, (bf16*)out_act, m, n, k, \
-                      lda, ldw, ldc, ld_act, mode, glu_kind, act_p, act_q)
+                      lda, ldw, ldc, ld_act, mode, glu_kind, act_p, act_q, add, second)
     if (m <= 8) { LAUNCH(1); }
     else if (m <= 16) { LAUNCH(2); }
     else if (m <= 32) { LAUNCH(4); }
@@ -237,6 +260,30 @@ extern "C" int ti_gemm_skinny_glu(const void* a, const void* w, void* out_act, i
                                   int ld_act, int glu_kind, float glu_limit, float glu_alpha, void* stream) {
     TI_REQUIRE(glu_kind >= GLU_SILU && glu_kind <= GLU_GELU_TANH, "gemm_skinny_glu: activation %d", glu_kind);
     return skinny(a, w, nullptr, out_act, m, n, k, lda, ldw, 0, ld_act, MODE_SWIGLU, glu_kind, glu_limit, glu_alpha, stream);
+}
+
+// c += scale sigmoid(gate + bias) * (a w^T), element by element; gate float32 [m, n] (row stride ld_gate), bias [n]
+extern "C" int ti_gemm_skinny_gated(const void* a, const void* w, float* c, int m, int n, int k, int lda, int ldw,
+                                    int ldc, const float* gate, int ld_gate, const float* bias, float scale,
+                                    void* stream) {
+    TI_REQUIRE(gate != nullptr && bias != nullptr, "gemm_skinny_gated: a gate and its bias");
+    return skinny(a, w, c, nullptr, m, n, k, lda, ldw, ldc, 0, MODE_ACCUMULATE, GLU_SILU, 0.0f, 0.0f, stream,
+                  AddGate{gate, ld_gate, bias, scale});
+}
+
+// Two products of m rows and the same k in one launch: the first stores its float32 rows into c, or (glu_kind >= 0)
+// its gated activation over strips of 8 and 8 into out_act; the second stores a2 w2^T into c2.
+extern "C" int ti_gemm_skinny_pair(const void* a, const void* w, float* c, void* out_act, int m, int n, int k, int lda,
+                                   int ldw, int ldc, int ld_act, int glu_kind, float glu_limit, float glu_alpha,
+                                   const void* a2, const void* w2, float* c2, int n2, int lda2, int ldw2, int ldc2,
+                                   void* stream) {
+    if (m == 0 || n == 0 || n2 == 0) return 0;
+    TI_REQUIRE(glu_kind <= GLU_GELU_TANH, "gemm_skinny_pair: activation %d", glu_kind);
+    TI_REQUIRE(ti_gemm_skinny_supported(m, n2, k, lda2, ldw2) && (uintptr_t)a2 % 16 == 0 && (uintptr_t)w2 % 16 == 0,
+               "gemm_skinny_pair: the second product's operands");
+    return skinny(a, w, c, out_act, m, n, k, lda, ldw, ldc, ld_act, glu_kind < 0 ? MODE_STORE : MODE_SWIGLU,
+                  glu_kind < 0 ? GLU_SILU : glu_kind, glu_limit, glu_alpha, stream, AddGate{nullptr, 0, nullptr, 0.0f},
+                  SecondProduct{(const bf16*)a2, (const bf16*)w2, c2, n2, lda2, ldw2, ldc2, 0});
 }
 
 // out_act[m, n] (bfloat16) = xielu(a w^T): act_p z^2 + z/2 for z > 0, act_q (exp(z) - 1 - z) + z/2 otherwise

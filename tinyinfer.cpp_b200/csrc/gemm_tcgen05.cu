@@ -11,7 +11,7 @@
 // warps 2-9 read a finished accumulator with tcgen05.ld (a warp reads the 32 TMEM lanes = rows
 // that its position in the warpgroup allows) and run the epilogue while the next tile's
 // products already fill the other accumulator.  Epilogues: store, accumulate into C (the
-// residual stream), SwiGLU over 8 gate + 8 up columns into bfloat16, or (BN = 256) the QKV
+// residual stream; optionally through a gate, C += scale sigmoid(gate + bias) * sum), SwiGLU over 8 gate + 8 up columns into bfloat16, or (BN = 256) the QKV
 // epilogue of qkv_epilogue.cuh: head norm, rotation and the store into the paged cache.  Rows and columns past
 // M, N and K are zero-filled by TMA on the way in and skipped on the way out.
 //
@@ -57,7 +57,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                     bf16* __restrict__ out_act, int m, int n, int k, int ldc, int ld_act, int mode,
                     float* __restrict__ ws, int splits, int* __restrict__ status,
                     const int* __restrict__ group_of_tile, const int* __restrict__ tiles_m_dev,
-                    const GluArgs glu) {
+                    const GluArgs glu, const AddGate add) {
     using T = Tile<BN>;
     constexpr int STAGES = T::STAGES;
     extern __shared__ unsigned char smem_raw[];
@@ -263,8 +263,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                                 was = *reinterpret_cast<const float4*>(dst + i);
                                 if (second) was2 = *reinterpret_cast<const float4*>(dst + i + 4);
                             }
-                            x.x += was.x; x.y += was.y; x.z += was.z; x.w += was.w;
-                            y.x += was2.x; y.y += was2.y; y.z += was2.z; y.w += was2.w;
+                            x = add_through4(add, row, col + i, was, x);
+                            if (second) y = add_through4(add, row, col + i + 4, was2, y);
                         }
                         if (by8) {
                             store_f32x8(dst + i, x, y);
@@ -307,7 +307,7 @@ __global__ void rope_table_kernel(const int* __restrict__ positions, const float
 // c (+)= the sum of the runs' slabs ws[run][m][n], in ascending order of the run (of K).
 __global__ void __launch_bounds__(256)
 gemm_split_merge_kernel(const float* ws, float* __restrict__ c, int m, int n, int ldc, int splits,
-                        int accumulate) {
+                        int accumulate, const AddGate add) {
     pdl_launch();
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;      // a float4 of the output
     const int n4 = n / 4;
@@ -323,8 +323,7 @@ gemm_split_merge_kernel(const float* ws, float* __restrict__ c, int m, int n, in
         const float4 v = __ldcg(reinterpret_cast<const float4*>(src + r * slab));
         sum.x += v.x; sum.y += v.y; sum.z += v.z; sum.w += v.w;
     }
-    *reinterpret_cast<float4*>(c + (size_t)row * ldc + col) =
-        make_float4(was.x + sum.x, was.y + sum.y, was.z + sum.z, was.w + sum.w);
+    *reinterpret_cast<float4*>(c + (size_t)row * ldc + col) = add_through4(add, row, col, was, sum);
 }
 
 constexpr int MAX_SPLITS = 8, MIN_RUN_KB = 4;
@@ -355,7 +354,8 @@ int choose_splits(int m, int n, int k, int mode, int sms) {
 // width: the tiles' columns, 256, 128 or 64
 int launch_tiles(const void* a, const void* w, const qkv::Epilogue& e, float* c, void* out_act, int m, int n,
                  int k, int lda, int ldw, int ldc, int ld_act, int mode, int width, float* ws, int splits,
-                 int* status, void* stream, bool add_runs = true, GluArgs glu = GluArgs{GLU_SILU, 0.0f, 0.0f}) {
+                 int* status, void* stream, bool add_runs = true, GluArgs glu = GluArgs{GLU_SILU, 0.0f, 0.0f},
+                 AddGate add = AddGate{nullptr, 0, nullptr, 0.0f}) {
     int device = 0, sms = 0;
     cudaGetDevice(&device);
     cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, device);
@@ -380,23 +380,23 @@ int launch_tiles(const void* a, const void* w, const qkv::Epilogue& e, float* c,
         const int tiles = tiles_m * ((n + 255) / 256) * splits;
         ti_launch_pdl(gemm_tcgen05_kernel<256>, tiles < sms ? tiles : sms, THREADS, Tile<256>::SMEM,
                       (cudaStream_t)stream, map_a, map_w, e, c, (bf16*)out_act, m, n, k, ldc, ld_act, mode, ws,
-                      splits, status, (const int*)nullptr, (const int*)nullptr, glu);
+                      splits, status, (const int*)nullptr, (const int*)nullptr, glu, add);
     } else if (width == 128) {
         const int tiles = tiles_m * ((n + 127) / 128) * splits;
         ti_launch_pdl(gemm_tcgen05_kernel<128>, tiles < sms ? tiles : sms, THREADS, Tile<128>::SMEM,
                       (cudaStream_t)stream, map_a, map_w, e, c, (bf16*)out_act, m, n, k, ldc, ld_act, mode, ws,
-                      splits, status, (const int*)nullptr, (const int*)nullptr, glu);
+                      splits, status, (const int*)nullptr, (const int*)nullptr, glu, add);
     } else {
         const int tiles = tiles_m * ((n + 63) / 64) * splits;
         ti_launch_pdl(gemm_tcgen05_kernel<64>, tiles < sms ? tiles : sms, THREADS, Tile<64>::SMEM,
                       (cudaStream_t)stream, map_a, map_w, e, c, (bf16*)out_act, m, n, k, ldc, ld_act, mode, ws,
-                      splits, status, (const int*)nullptr, (const int*)nullptr, glu);
+                      splits, status, (const int*)nullptr, (const int*)nullptr, glu, add);
     }
     if (int rc = ti_check_launch("gemm_tcgen05")) return rc;
     if (splits > 1 && add_runs) {
         const long long quads = (long long)m * (n / 4);
         ti_launch_pdl(gemm_split_merge_kernel, (unsigned)((quads + 255) / 256), 256, 0, (cudaStream_t)stream,
-                      (const float*)ws, c, m, n, ldc, splits, mode == MODE_ACCUMULATE ? 1 : 0);
+                      (const float*)ws, c, m, n, ldc, splits, mode == MODE_ACCUMULATE ? 1 : 0, add);
         return ti_check_launch("gemm_split_merge");
     }
     return 0;
@@ -427,7 +427,7 @@ extern "C" int ti_gemm_tcgen05_add_runs(const float* ws, float* c, int m, int n,
                "gemm_tcgen05_add_runs: N=%d and the row stride %d must be multiples of 4", n, ldc);
     const long long quads = (long long)m * (n / 4);
     ti_launch_pdl(gemm_split_merge_kernel, (unsigned)((quads + 255) / 256), 256, 0, (cudaStream_t)stream, ws, c, m,
-                  n, ldc, runs, accumulate ? 1 : 0);
+                  n, ldc, runs, accumulate ? 1 : 0, AddGate{nullptr, 0, nullptr, 0.0f});
     return ti_check_launch("gemm_split_merge");
 }
 
@@ -435,9 +435,8 @@ extern "C" int ti_gemm_tcgen05_add_runs(const float* ws, float* c, int m, int n,
 // ws: null, or the scratch for ti_gemm_tcgen05_splits(m, n, k, mode) runs of K (16-byte aligned).
 // leave_runs: with K cut, do not add the runs into c; the caller does (ti_gemm_tcgen05_add_runs, or
 // a norm that completes its rows from the slabs).
-extern "C" int ti_gemm_tcgen05(const void* a, const void* w, float* c, void* out_act, int m, int n,
-                               int k, int lda, int ldw, int ldc, int ld_act, int mode, float* ws,
-                               int leave_runs, int* status, void* stream) {
+static int gemm_tcgen05(const void* a, const void* w, float* c, void* out_act, int m, int n, int k, int lda, int ldw,
+                        int ldc, int ld_act, int mode, float* ws, int leave_runs, int* status, void* stream, AddGate add) {
     if (m == 0 || n == 0) return 0;
     TI_REQUIRE(mode >= MODE_STORE && mode <= MODE_SWIGLU, "gemm_tcgen05: mode %d", mode);
     TI_REQUIRE(ti_gemm_tcgen05_supported(m, n, k, lda, ldw, ldc, mode),
@@ -457,11 +456,29 @@ extern "C" int ti_gemm_tcgen05(const void* a, const void* w, float* c, void* out
     if (splits > 1) {
         TI_REQUIRE((uintptr_t)ws % 16 == 0, "gemm_tcgen05: the scratch must be 16-byte aligned");
         return launch_tiles(a, w, qkv::Epilogue{}, c, out_act, m, n, k, lda, ldw, ldc, ld_act, mode, 128, ws,
-                            splits, status, stream, !leave_runs);
+                            splits, status, stream, !leave_runs, GluArgs{GLU_SILU, 0.0f, 0.0f}, add);
     }
     const int width = tiles_m * ((n + 255) / 256) >= sms ? 256 : tiles_m * ((n + 127) / 128) * 2 >= sms ? 128 : 64;
     return launch_tiles(a, w, qkv::Epilogue{}, c, out_act, m, n, k, lda, ldw, ldc, ld_act, mode, width, nullptr, 1,
-                        status, stream);
+                        status, stream, true, GluArgs{GLU_SILU, 0.0f, 0.0f}, add);
+}
+
+extern "C" int ti_gemm_tcgen05(const void* a, const void* w, float* c, void* out_act, int m, int n,
+                               int k, int lda, int ldw, int ldc, int ld_act, int mode, float* ws,
+                               int leave_runs, int* status, void* stream) {
+    return gemm_tcgen05(a, w, c, out_act, m, n, k, lda, ldw, ldc, ld_act, mode, ws, leave_runs, status, stream,
+                        AddGate{nullptr, 0, nullptr, 0.0f});
+}
+
+// c += scale sigmoid(gate + bias) * (a w^T), element by element; gate float32 [m, n] (row stride ld_gate), bias [n],
+// both on 16 bytes; the runs of a cut K pass the gate in the launch that adds them
+extern "C" int ti_gemm_tcgen05_gated(const void* a, const void* w, float* c, int m, int n, int k, int lda, int ldw,
+                                     int ldc, float* ws, const float* gate, int ld_gate, const float* bias, float scale,
+                                     int* status, void* stream) {
+    TI_REQUIRE((uintptr_t)gate % 16 == 0 && (uintptr_t)bias % 16 == 0 && ld_gate % 4 == 0 && gate != nullptr && bias != nullptr,
+               "gemm_tcgen05_gated: the gate's rows and the bias must start on 16 bytes");
+    return gemm_tcgen05(a, w, c, nullptr, m, n, k, lda, ldw, ldc, 0, MODE_ACCUMULATE, ws, 0, status, stream,
+                        AddGate{gate, ld_gate, bias, scale});
 }
 
 // Grouped product: row tile i (128 rows of a) is multiplied by the i-th named group's weights,
@@ -503,11 +520,11 @@ static int gemm_tcgen05_grouped_impl(const void* a, const void* w, float* c, voi
     if (width == 256)
         gemm_tcgen05_kernel<256><<<grid, THREADS, Tile<256>::SMEM, (cudaStream_t)stream>>>(
             map_a, map_w, qkv::Epilogue{}, c, (bf16*)out_act, m_max, n, k, ldc, ld_act, mode, nullptr, 1, status,
-            group_of_tile, tiles_m_dev, glu);
+            group_of_tile, tiles_m_dev, glu, AddGate{nullptr, 0, nullptr, 0.0f});
     else
         gemm_tcgen05_kernel<128><<<grid, THREADS, Tile<128>::SMEM, (cudaStream_t)stream>>>(
             map_a, map_w, qkv::Epilogue{}, c, (bf16*)out_act, m_max, n, k, ldc, ld_act, mode, nullptr, 1, status,
-            group_of_tile, tiles_m_dev, glu);
+            group_of_tile, tiles_m_dev, glu, AddGate{nullptr, 0, nullptr, 0.0f});
     return ti_check_launch("gemm_tcgen05_grouped");
 }
 

@@ -16,6 +16,7 @@
 // leader.  Every wait is bounded; on a timeout the block records status 2 and both blocks leave
 // through the cluster barrier at the end, freeing their tensor memory.
 #include "qkv_epilogue.cuh"
+#include "glu.cuh"
 
 namespace {
 
@@ -85,7 +86,7 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(THREADS, 1)
 gemm_tcgen05_2sm_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
                         const __grid_constant__ qkv::Epilogue qkv_e, float* __restrict__ c,
                         bf16* __restrict__ out_act, int m, int n, int k, int ldc, int ld_act, int mode,
-                        int* __restrict__ status) {
+                        int* __restrict__ status, const AddGate add) {
     constexpr int STAGES = Pair<BN>::STAGES, STAGE_B = Pair<BN>::STAGE_B;
     constexpr unsigned TMEM_COLS = Pair<BN>::TMEM_COLS;
     extern __shared__ unsigned char smem_raw[];
@@ -240,12 +241,8 @@ gemm_tcgen05_2sm_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
                         float4 y = make_float4(v[i + 4], v[i + 5], v[i + 6], v[i + 7]);
                         const bool second = col + i + 4 < n;
                         if (mode == MODE_ACCUMULATE) {
-                            const float4 old = *reinterpret_cast<const float4*>(dst + i);
-                            x.x += old.x; x.y += old.y; x.z += old.z; x.w += old.w;
-                            if (second) {
-                                const float4 old2 = *reinterpret_cast<const float4*>(dst + i + 4);
-                                y.x += old2.x; y.y += old2.y; y.z += old2.z; y.w += old2.w;
-                            }
+                            x = add_through4(add, row, col + i, *reinterpret_cast<const float4*>(dst + i), x);
+                            if (second) y = add_through4(add, row, col + i + 4, *reinterpret_cast<const float4*>(dst + i + 4), y);
                         }
                         if (by8) {
                             store_f32x8(dst + i, x, y);
@@ -282,7 +279,8 @@ extern "C" int ti_gemm_tcgen05_2sm_supported(int m, int n, int k, int lda, int l
 namespace {
 
 int launch_pairs(const void* a, const void* w, const qkv::Epilogue& e, float* c, void* out_act, int m, int n,
-                 int k, int lda, int ldw, int ldc, int ld_act, int mode, int* status, void* stream) {
+                 int k, int lda, int ldw, int ldc, int ld_act, int mode, int* status, void* stream,
+                 AddGate add = AddGate{nullptr, 0, nullptr, 0.0f}) {
     int device = 0, sms = 0;
     cudaGetDevice(&device);
     cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, device);
@@ -299,7 +297,7 @@ int launch_pairs(const void* a, const void* w, const qkv::Epilogue& e, float* c,
     const int tiles = ((m + BM - 1) / BM) * ((n + 255) / 256);
     const int pairs = tiles < sms / 2 ? tiles : sms / 2;
     ti_launch_pdl(gemm_tcgen05_2sm_kernel<256>, 2 * pairs, THREADS, Pair<256>::SMEM, (cudaStream_t)stream,
-                  map_a, map_w, e, c, (bf16*)out_act, m, n, k, ldc, ld_act, mode, status);
+                  map_a, map_w, e, c, (bf16*)out_act, m, n, k, ldc, ld_act, mode, status, add);
     return ti_check_launch("gemm_tcgen05_2sm");
 }
 
@@ -319,6 +317,21 @@ extern "C" int ti_gemm_tcgen05_2sm(const void* a, const void* w, float* c, void*
     TI_REQUIRE(mode == MODE_SWIGLU ? ((uintptr_t)out_act % 16 == 0 && ld_act % 8 == 0) : (uintptr_t)c % 16 == 0,
                "gemm_tcgen05_2sm: the output must be 16-byte aligned");
     return launch_pairs(a, w, qkv::Epilogue{}, c, out_act, m, n, k, lda, ldw, ldc, ld_act, mode, status, stream);
+}
+
+// c += scale sigmoid(gate + bias) * (a w^T): as ti_gemm_tcgen05_gated, K never cut
+extern "C" int ti_gemm_tcgen05_2sm_gated(const void* a, const void* w, float* c, int m, int n, int k, int lda, int ldw,
+                                         int ldc, const float* gate, int ld_gate, const float* bias, float scale,
+                                         int* status, void* stream) {
+    if (m == 0 || n == 0) return 0;
+    TI_REQUIRE(ti_gemm_tcgen05_2sm_supported(m, n, k, lda, ldw, ldc, MODE_ACCUMULATE),
+               "gemm_tcgen05_2sm_gated: K=%d and the row strides %d, %d must be multiples of 8, N=%d a multiple of 4", k, lda,
+               ldw, n);
+    TI_REQUIRE((uintptr_t)a % 16 == 0 && (uintptr_t)w % 16 == 0 && (uintptr_t)c % 16 == 0 && (uintptr_t)gate % 16 == 0 &&
+               (uintptr_t)bias % 16 == 0 && ld_gate % 4 == 0 && gate != nullptr && bias != nullptr,
+               "gemm_tcgen05_2sm_gated: operands, output, the gate's rows and the bias must start on 16 bytes");
+    return launch_pairs(a, w, qkv::Epilogue{}, c, nullptr, m, n, k, lda, ldw, ldc, 0, MODE_ACCUMULATE, status, stream,
+                        AddGate{gate, ld_gate, bias, scale});
 }
 
 // The QKV product of a prompt portion with the epilogue of qkv_epilogue.cuh (head size 128):

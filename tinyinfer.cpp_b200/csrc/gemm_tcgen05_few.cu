@@ -18,6 +18,7 @@
 // accumulators with tcgen05.ld.  Every wait on an mbarrier is bounded: on a timeout the block
 // records status 2, frees its tensor memory and returns.
 #include "sm100.cuh"
+#include "glu.cuh"
 
 namespace {
 
@@ -58,7 +59,8 @@ struct Units {
 
 // 16 tokens' values of W row `n_row` (this thread's), tokens tok0 .. tok0 + 15.
 __device__ __forceinline__ void finish16(const float (&v)[16], int tok0, int n_row, int lane, float* c,
-                                         bf16* out_act, int m, int n, int ldc, int ld_act, int mode) {
+                                         bf16* out_act, int m, int n, int ldc, int ld_act, int mode,
+                                         const AddGate& add) {
     if (mode == MODE_SWIGLU) {
         // rows of W: 8 gate, their 8 up, ...; lane l (l % 16 < 8) holds a gate row, lane l + 8 its up row
 #pragma unroll
@@ -75,7 +77,11 @@ __device__ __forceinline__ void finish16(const float (&v)[16], int tok0, int n_r
         // one after the other, every read would wait behind the store before it (the compiler
         // cannot tell that the addresses differ), a round trip to L2 per row (the down projection
         // of the 8B shape at 64 rows: 55 -> 34 microseconds).
-        float old[16];
+        float old[16], gate[16];
+        const float bias = add.gate ? add.bias[n_row] : 0.0f;
+#pragma unroll
+        for (int i = 0; i < 16; ++i)
+            gate[i] = add.gate && tok0 + i < m ? __ldcg(add.gate + (size_t)(tok0 + i) * add.ld + n_row) : 0.0f;
 #pragma unroll
         for (int i = 0; i < 16; ++i)
             old[i] = mode == MODE_ACCUMULATE && tok0 + i < m ? __ldcg(c + (size_t)(tok0 + i) * ldc + n_row) : 0.0f;
@@ -83,7 +89,7 @@ __device__ __forceinline__ void finish16(const float (&v)[16], int tok0, int n_r
         for (int i = 0; i < 16; ++i) {
             const int tok = tok0 + i;
             if (tok >= m) break;
-            c[(size_t)tok * ldc + n_row] = old[i] + v[i];
+            c[(size_t)tok * ldc + n_row] = add_through(add, old[i], v[i], gate[i], bias);
         }
     }
 }
@@ -93,7 +99,7 @@ __global__ void __launch_bounds__(THREADS, BLOCKS_PER_SM)
 gemm_few_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
                 float* __restrict__ c, bf16* __restrict__ out_act, float* __restrict__ ws,
                 int* __restrict__ tickets, int m, int n, int k, int ldc, int ld_act, int mode, int splits,
-                int* __restrict__ status) {
+                int* __restrict__ status, const AddGate add) {
     using T = Few<NTOK>;
     constexpr int STAGES = T::STAGES;
     extern __shared__ unsigned char smem_raw[];
@@ -203,7 +209,7 @@ gemm_few_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
                 float v[16];
                 tmem_load16(tmem_base + ((unsigned)(quarter * 32) << 16) + (unsigned)(buf * NTOK + t0), v);
                 if (splits == 1) {
-                    finish16(v, t0, n_row, lane, c, out_act, m, n, ldc, ld_act, mode);
+                    finish16(v, t0, n_row, lane, c, out_act, m, n, ldc, ld_act, mode, add);
                 } else if (t0 < m) {
 #pragma unroll
                     for (int i = 0; i < 16; ++i) part[(size_t)(t0 + i) * BW + row_in_tile] = v[i];
@@ -250,7 +256,7 @@ gemm_few_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
             for (int t0 = 0; t0 < NTOK; t0 += 16) {
                 if (t0 < m)
                     finish16(*reinterpret_cast<const float(*)[16]>(&acc[t0]), t0, n_row, lane, c, out_act, m, n,
-                             ldc, ld_act, mode);
+                             ldc, ld_act, mode, add);
             }
             if (warp == 2 && lane == 0) tickets[tile] = 0;
         }
@@ -291,7 +297,7 @@ int device_sms() {
 template <int NTOK>
 int launch_few(const CUtensorMap& map_w, const CUtensorMap& map_x, float* c, bf16* out_act, float* ws,
                int* tickets, int m, int n, int k, int ldc, int ld_act, int mode, int splits, int sms,
-               int* status, cudaStream_t stream) {
+               int* status, cudaStream_t stream, AddGate add) {
     static TiPerDevice configured;
     if (configured.first_use()) {
         cudaError_t e = cudaFuncSetAttribute(gemm_few_kernel<NTOK>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -303,7 +309,7 @@ int launch_few(const CUtensorMap& map_w, const CUtensorMap& map_x, float* c, bf1
     const int slots = sms * BLOCKS_PER_SM;
     cudaError_t e = ti_launch_pdl(gemm_few_kernel<NTOK>, dim3(units < slots ? units : slots), dim3(THREADS),
                                   Few<NTOK>::SMEM, stream, map_w, map_x, c, out_act, ws, tickets, m, n, k, ldc,
-                                  ld_act, mode, splits, status);
+                                  ld_act, mode, splits, status, add);
     if (e != cudaSuccess) return ti_fail("gemm_tcgen05_few: %s", cudaGetErrorString(e));
     return ti_check_launch("gemm_tcgen05_few");
 }
@@ -326,9 +332,8 @@ extern "C" int ti_gemm_tcgen05_few_scratch(int m, int n, int k, long long* ws_fl
 }
 
 // mode 0: c = a w^T; 1: c += a w^T; 2: out_act[m, n/2] = SwiGLU over groups of 8 gate + 8 up rows of w.
-extern "C" int ti_gemm_tcgen05_few(const void* a, const void* w, float* c, void* out_act, int m, int n,
-                                   int k, int lda, int ldw, int ldc, int ld_act, int mode, float* ws,
-                                   int* tickets, int* status, void* stream) {
+static int few(const void* a, const void* w, float* c, void* out_act, int m, int n, int k, int lda, int ldw, int ldc,
+               int ld_act, int mode, float* ws, int* tickets, int* status, void* stream, AddGate add) {
     if (m == 0 || n == 0) return 0;
     TI_REQUIRE(ti_gemm_tcgen05_few_supported(m, n, k, lda, ldw, mode),
                "gemm_tcgen05_few: M=%d (1..64), K=%d and the row strides %d, %d (multiples of 8) or N=%d "
@@ -343,8 +348,24 @@ extern "C" int ti_gemm_tcgen05_few(const void* a, const void* w, float* c, void*
     if (int rc = make_map_bf16(&map_x, a, m, k, lda, ntok, "gemm_tcgen05_few")) return rc;
     cudaStream_t s = (cudaStream_t)stream;
     if (ntok == 16)
-        return launch_few<16>(map_w, map_x, c, (bf16*)out_act, ws, tickets, m, n, k, ldc, ld_act, mode, splits, sms, status, s);
+        return launch_few<16>(map_w, map_x, c, (bf16*)out_act, ws, tickets, m, n, k, ldc, ld_act, mode, splits, sms, status, s, add);
     if (ntok == 32)
-        return launch_few<32>(map_w, map_x, c, (bf16*)out_act, ws, tickets, m, n, k, ldc, ld_act, mode, splits, sms, status, s);
-    return launch_few<64>(map_w, map_x, c, (bf16*)out_act, ws, tickets, m, n, k, ldc, ld_act, mode, splits, sms, status, s);
+        return launch_few<32>(map_w, map_x, c, (bf16*)out_act, ws, tickets, m, n, k, ldc, ld_act, mode, splits, sms, status, s, add);
+    return launch_few<64>(map_w, map_x, c, (bf16*)out_act, ws, tickets, m, n, k, ldc, ld_act, mode, splits, sms, status, s, add);
+}
+
+extern "C" int ti_gemm_tcgen05_few(const void* a, const void* w, float* c, void* out_act, int m, int n, int k, int lda,
+                                   int ldw, int ldc, int ld_act, int mode, float* ws, int* tickets, int* status,
+                                   void* stream) {
+    return few(a, w, c, out_act, m, n, k, lda, ldw, ldc, ld_act, mode, ws, tickets, status, stream,
+               AddGate{nullptr, 0, nullptr, 0.0f});
+}
+
+// c += scale sigmoid(gate + bias) * (a w^T), element by element; gate float32 [m, n] (row stride ld_gate), bias [n]
+extern "C" int ti_gemm_tcgen05_few_gated(const void* a, const void* w, float* c, int m, int n, int k, int lda, int ldw,
+                                         int ldc, float* ws, int* tickets, const float* gate, int ld_gate,
+                                         const float* bias, float scale, int* status, void* stream) {
+    TI_REQUIRE(gate != nullptr && bias != nullptr, "gemm_tcgen05_few_gated: a gate and its bias");
+    return few(a, w, c, nullptr, m, n, k, lda, ldw, ldc, 0, MODE_ACCUMULATE, ws, tickets, status, stream,
+               AddGate{gate, ld_gate, bias, scale});
 }

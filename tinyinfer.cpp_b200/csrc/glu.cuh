@@ -15,6 +15,22 @@ __device__ __forceinline__ float gated_sum(float x, float y, float g, float scal
     return fmaf(scale / (1.0f + expf(-g)), y, x);
 }
 
+// What an epilogue that adds to C needs to know of such a gate (gate null: the plain sum).  `gate` is written by a
+// kernel of the same chain, so it is no read-only data.
+struct AddGate { const float* gate; int ld; const float* bias; float scale; };
+
+__device__ __forceinline__ float add_through(const AddGate& g, float was, float y, float gate, float bias) {
+    return g.gate ? gated_sum(was, y, gate + bias, g.scale) : was + y;
+}
+// four neighbouring columns (row, col .. col + 3); the gate's rows and the bias start on 16 bytes
+__device__ __forceinline__ float4 add_through4(const AddGate& g, int row, int col, float4 was, float4 y) {
+    if (g.gate == nullptr) return make_float4(was.x + y.x, was.y + y.y, was.z + y.z, was.w + y.w);
+    const float4 v = __ldcg(reinterpret_cast<const float4*>(g.gate + (size_t)row * g.ld + col));
+    const float4 b = __ldg(reinterpret_cast<const float4*>(g.bias + col));
+    return make_float4(gated_sum(was.x, y.x, v.x + b.x, g.scale), gated_sum(was.y, y.y, v.y + b.y, g.scale),
+                       gated_sum(was.z, y.z, v.z + b.z, g.scale), gated_sum(was.w, y.w, v.w + b.w, g.scale));
+}
+
 // gelu(z) = z/2 (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))
 __device__ __forceinline__ float gelu_tanh(float z) {
     const float inner = 0.7978845608028654f * fmaf(0.044715f * z * z, z, z);

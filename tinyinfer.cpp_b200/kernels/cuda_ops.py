@@ -178,6 +178,11 @@ class CudaOps(MixerOps, StateOps):
         # ... and with the product in front of it that adds to the same residual (a mixer's output
         # projection, asked for with ``linear(..., may_defer=True)``) and the norm between them
         self.fuse_decode_tail = True
+        # two products of few rows that read the same step's rows and depend on nothing of each other
+        # (``linear(..., may_pair=True)`` and the product after it) as one launch
+        self.pair_few_rows = True
+        self.fuse_gated_sums = True       # a gate on the way into the residual in the product's epilogue
+        self._pending_pair = None         # (a, w, out) of a product that waits for the next one
         self._ffn_counters = None
         self._pending = None              # a held-back ``out += a w^T`` (and the norm of ``out`` after it)
         self._retired = []                # outgrown counter buffers that captured graphs may still use
@@ -229,6 +234,11 @@ class CudaOps(MixerOps, StateOps):
             b.ti_gemm_skinny.argtypes = [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp]
             b.ti_gemm_skinny_supported.argtypes = [_i, _i, _i, _i, _i]
             b.ti_gemm_skinny_xielu.argtypes = [_vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _f, _vp]
+            b.ti_gemm_skinny_gated.argtypes = [_vp, _vp, _vp] + [_i] * 6 + [_vp, _i, _vp, _f, _vp]
+            b.ti_gemm_skinny_pair.argtypes = [_vp, _vp, _vp, _vp] + [_i] * 8 + [_f, _f, _vp, _vp, _vp] + [_i] * 4 + [_vp]
+            b.ti_gemm_tcgen05_few_gated.argtypes = [_vp, _vp, _vp] + [_i] * 6 + [_vp, _vp, _vp, _i, _vp, _f, _vp, _vp]
+            b.ti_gemm_tcgen05_gated.argtypes = [_vp, _vp, _vp] + [_i] * 6 + [_vp, _vp, _i, _vp, _f, _vp, _vp]
+            b.ti_gemm_tcgen05_2sm_gated.argtypes = [_vp, _vp, _vp] + [_i] * 6 + [_vp, _i, _vp, _f, _vp, _vp]
             b.ti_ffn_decode_supported.argtypes = [_i] * 8
             b.ti_ffn_decode.argtypes = [_vp, _vp, _vp, _vp, _vp] + [_i] * 8 + [_vp, _vp, _vp]
             b.ti_attn_out_ffn_decode_supported.argtypes = [_i] * 10
@@ -380,19 +390,28 @@ class CudaOps(MixerOps, StateOps):
         elif runs > 1:
             self.launches += 1            # the launch that adds the runs
 
-    def _few_tc(self, a, w, c, out_act, mode) -> bool:
-        """Runs the split-K tcgen05 product for few rows if it applies to these operands."""
+    def _few_tc_scratch(self, a, w, mode):
+        """Workspace (or None) and tickets of the split-K tcgen05 product for few rows, or None if it does
+        not apply to these operands."""
         m, k = a.shape
         n = w.shape[0]
         if (self.few_tc_min_bytes is None or m > 64 or n * k * 2 <= self.few_tc_min_bytes
                 or a.data_ptr() % 16 or w.data_ptr() % 16
                 or not self.bf16.ti_gemm_tcgen05_few_supported(m, n, k, a.stride(0), w.stride(0), mode)):
-            return False
+            return None
         ws_floats, tickets = ctypes.c_longlong(0), ctypes.c_int(0)
         self.bf16.ti_gemm_tcgen05_few_scratch(m, n, k, ctypes.byref(ws_floats), ctypes.byref(tickets))
         if self._few_tickets is None or self._few_tickets.numel() < tickets.value:
             self._few_tickets = self._grown(self._few_tickets, tickets.value, a.device)
         ws = torch.empty(ws_floats.value, dtype=torch.float32, device=a.device) if ws_floats.value else None
+        return ws, self._few_tickets
+
+    def _few_tc(self, a, w, c, out_act, mode) -> bool:
+        """Runs the split-K tcgen05 product for few rows if it applies to these operands."""
+        scratch = self._few_tc_scratch(a, w, mode)
+        if scratch is None:
+            return False
+        ws, m, k, n = scratch[0], a.shape[0], a.shape[1], w.shape[0]
         self._ok(self.bf16.ti_gemm_tcgen05_few(
             a.data_ptr(), w.data_ptr(), _ptr(c), _ptr(out_act), m, n, k, a.stride(0), w.stride(0),
             c.stride(0) if c is not None else 0, out_act.stride(0) if out_act is not None else 0, mode,
@@ -469,7 +488,11 @@ class CudaOps(MixerOps, StateOps):
                                                     c.stride(0), runs, int(accumulate), self._stream()), self.bf16)
 
     def flush(self) -> None:
-        """Launch what ``linear(..., may_defer=True)`` and a norm after it have held back."""
+        """Launch what ``linear(..., may_defer=True)`` and a norm after it, or ``linear(..., may_pair=True)``,
+        have held back."""
+        held, self._pending_pair = self._pending_pair, None
+        if held is not None:
+            self.linear(*held)
         pr, self._pending_runs = self._pending_runs, None
         if pr is not None:
             self._add_runs(pr)
@@ -481,13 +504,46 @@ class CudaOps(MixerOps, StateOps):
             weight, eps, normed = p["norm"]
             self.rmsnorm(p["out"], weight, eps, normed)
 
-    def linear(self, a, w, out, accumulate=False, may_defer=False):
+    def _pairable(self, a, w) -> bool:
+        """Whether the few-row product that streams the weights once takes these operands."""
+        m, k = a.shape
+        n = w.shape[0]
+        return (a.dtype == w.dtype == torch.bfloat16 and a.stride(1) == w.stride(1) == 1 and a.data_ptr() % 16 == 0
+                and w.data_ptr() % 16 == 0 and w.shape[1] == k
+                and (self.few_tc_min_bytes is None or n * k * 2 <= self.few_tc_min_bytes)
+                and bool(self.bf16.ti_gemm_skinny_supported(m, n, k, a.stride(0), w.stride(0))))
+
+    def _launch_pair(self, a, w, out, out_act, glu=None) -> bool:
+        """Runs the product that ``may_pair`` held back beside this one, if the two fit one launch."""
+        held = self._pending_pair
+        if held is None:
+            return False
+        a2, w2, out2 = held
+        m, k = a.shape
+        if a2.shape != a.shape or not (glu is not None or self._pairable(a, w)):
+            return False
+        self._pending_pair = None
+        kind, limit, alpha = glu if glu is not None else (-1, 0.0, 0.0)
+        self._ok(self.bf16.ti_gemm_skinny_pair(
+            a.data_ptr(), w.data_ptr(), _ptr(out), _ptr(out_act), m, w.shape[0], k, a.stride(0), w.stride(0),
+            out.stride(0) if out is not None else 0, out_act.stride(0) if out_act is not None else 0, kind, float(limit),
+            float(alpha), a2.data_ptr(), w2.data_ptr(), out2.data_ptr(), w2.shape[0], a2.stride(0), w2.stride(0),
+            out2.stride(0), self._stream()), self.bf16)
+        return True
+
+    def linear(self, a, w, out, accumulate=False, may_defer=False, may_pair=False):
         """out (+)= a @ w.T.  With ``may_defer`` (and ``accumulate``) the kernel set may hold the
         product back and run it in one launch with a norm of ``out`` and a feed-forward into ``out``
         that follow immediately; any other operation of the kernel set, ``stream()`` and
         ``flush()`` launch it first.  The caller must not touch ``a`` or ``out`` by other means
-        until then.  ``out`` may be a ``parts.base.GatedSum`` (with ``accumulate``): the product then
+        until then.  With ``may_pair`` (a plain store) a product of few rows may wait for the next one
+        and share its launch; it too is launched by ``flush()`` at the latest.  ``out`` may be a ``parts.base.GatedSum`` (with ``accumulate``): the product then
         passes that gate on its way into the residual."""
+        if self._pending_pair is not None:
+            if (not accumulate and isinstance(out, torch.Tensor) and out.dtype == torch.float32 and out.stride(1) == 1
+                    and tuple(out.shape) == (a.shape[0], w.shape[0]) and self._launch_pair(a, w, out, None)):
+                return
+            self.flush()
         if self._pending is not None or self._pending_runs is not None:
             self.flush()
         if not isinstance(out, torch.Tensor):
@@ -501,6 +557,10 @@ class CudaOps(MixerOps, StateOps):
                 and w.shape[1] == k and tuple(out.shape) == (m, n)
                 and a.stride(1) == w.stride(1) == out.stride(1) == 1):
             self._pending = {"a": a, "w": w, "out": out}
+            return
+        if (may_pair and self.pair_few_rows and not accumulate and out.dtype == torch.float32 and out.stride(1) == 1
+                and tuple(out.shape) == (m, n) and self._pairable(a, w)):
+            self._pending_pair = (a, w, out)
             return
         _need(w.shape[1] == k and tuple(out.shape) == (m, n), "linear: shapes do not agree")
         _need(out.dtype == torch.float32, "linear: out must be float32")
@@ -526,7 +586,39 @@ class CudaOps(MixerOps, StateOps):
             self._stream()))
 
     def _linear_gated_sum(self, a, w, target):
-        """``x += scale * sigmoid(gate + bias) * (a @ w.T)`` for a ``parts.base.GatedSum``."""
+        """``x += scale * sigmoid(gate + bias) * (a @ w.T)`` for a ``parts.base.GatedSum``: in the product's
+        epilogue where a tensor-core product takes the operands, else behind it."""
+        x, gate, bias = target.x, target.gate, target.bias
+        m, k = a.shape
+        n = w.shape[0]
+        _need(w.shape[1] == k and tuple(x.shape) == tuple(gate.shape) == (m, n) and bias.numel() == n
+              and x.dtype == gate.dtype == bias.dtype == torch.float32 and bias.is_contiguous()
+              and x.stride(1) == gate.stride(1) == 1, "linear: a gated sum of float32 rows of the product's shape")
+        if (self.fuse_gated_sums and a.dtype == w.dtype == torch.bfloat16 and a.stride(1) == w.stride(1) == 1
+                and a.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0):
+            args = (gate.data_ptr(), gate.stride(0), bias.data_ptr(), float(target.scale))
+            sizes = (a.data_ptr(), w.data_ptr(), x.data_ptr(), m, n, k, a.stride(0), w.stride(0), x.stride(0))
+            status, stream = self.status.data_ptr(), self._stream()
+            few = self._few_tc_scratch(a, w, 1)
+            if few is not None:
+                self._ok(self.bf16.ti_gemm_tcgen05_few_gated(*sizes, _ptr(few[0]), few[1].data_ptr(), *args, status, stream),
+                         self.bf16)
+                return
+            if self.bf16.ti_gemm_skinny_supported(m, n, k, a.stride(0), w.stride(0)):
+                self._ok(self.bf16.ti_gemm_skinny_gated(*sizes, *args, stream), self.bf16)
+                return
+            if (m > 64 and x.data_ptr() % 16 == 0 and gate.data_ptr() % 16 == 0 and gate.stride(0) % 4 == 0
+                    and bias.data_ptr() % 16 == 0
+                    and self.bf16.ti_gemm_tcgen05_supported(m, n, k, a.stride(0), w.stride(0), x.stride(0), 1)):
+                if self._tc_gemm(m, n) is self.bf16.ti_gemm_tcgen05_2sm:
+                    self._ok(self.bf16.ti_gemm_tcgen05_2sm_gated(*sizes, *args, status, stream), self.bf16)
+                    return
+                runs = int(self.bf16.ti_gemm_tcgen05_splits(m, n, k, 1)) if self.split_k_portions else 1
+                ws = torch.empty(runs * m * n, dtype=torch.float32, device=a.device) if runs > 1 else None
+                self._ok(self.bf16.ti_gemm_tcgen05_gated(*sizes, _ptr(ws), *args, status, stream), self.bf16)
+                if runs > 1:
+                    self.launches += 1        # the launch that adds the runs
+                return
         y = torch.empty((a.shape[0], w.shape[0]), dtype=torch.float32, device=a.device)
         self.linear(a, w, y)
         self.gated_add(y, target)
@@ -589,9 +681,11 @@ class CudaOps(MixerOps, StateOps):
                 and h.data_ptr() % 16 == 0
                 and self.bf16.ti_gemm_skinny_supported(m, 2 * inter, k, h.stride(0), w_gate_up.stride(0))):
             # few rows: the activation in the epilogue of the product that streams the weights once
-            self._ok(self.bf16.ti_gemm_skinny_glu(
-                h.data_ptr(), w_gate_up.data_ptr(), y.data_ptr(), m, 2 * inter, k, h.stride(0), w_gate_up.stride(0),
-                y.stride(0), GLU_KINDS[kind], float(limit), float(alpha), self._stream()), self.bf16)
+            if not self._launch_pair(h, w_gate_up, None, y, (GLU_KINDS[kind], limit, alpha)):
+                self.flush()
+                self._ok(self.bf16.ti_gemm_skinny_glu(
+                    h.data_ptr(), w_gate_up.data_ptr(), y.data_ptr(), m, 2 * inter, k, h.stride(0), w_gate_up.stride(0),
+                    y.stride(0), GLU_KINDS[kind], float(limit), float(alpha), self._stream()), self.bf16)
         elif (interleaved and m > 64 and h.dtype == torch.bfloat16 and w_gate_up.dtype == torch.bfloat16
                 and inter % 8 == 0 and h.data_ptr() % 16 == 0 and self.bf16.ti_gemm_tcgen05_supported(
                     m, 2 * inter, k, h.stride(0), w_gate_up.stride(0), 0, 2)):

@@ -228,6 +228,7 @@ class StateOps:
     # ---- sums that pass a gate ---------------------------------------------------------------------
     def gated_add(self, y, target):
         """``x += scale * sigmoid(gate + bias) * y`` for a ``parts.base.GatedSum`` ``target``."""
+        self.flush()
         x, gate, bias = target.x, target.gate, target.bias
         for v in (x, gate, y):
             self._want(v.dtype == torch.float32 and v.stride(1) == 1 and tuple(v.shape) == tuple(x.shape),

@@ -85,7 +85,7 @@ class GatedPreNormBlock(Part):
         """``x += m sigmoid(Wg h + b) * part(.)``; ``run(target)`` lets the part add its result to ``target``."""
         w, bias = gate
         g = torch.empty_like(x)
-        ops.linear(h, w, g)
+        ops.linear(h, w, g, may_pair=True)
         target = GatedSum(x, g, bias, self.multiplier)
         if part.ends_in_linear:
             run(target)
