@@ -106,16 +106,19 @@ template <int VPT, int LANES> __device__ __forceinline__ float lanes_sum(const f
 
 // Small blocks of cut columns share an SM (the registers of at least 768 threads fit), so that other warps issue
 // while one waits on its sums.
-template <int MODE, int CB, int LANES> struct StateBlock {
+template <int MODE, int DMAX, int CB, int LANES> struct StateBlock {
     // columns a thread holds (a k or q read serves them all): two for the cut columns halved the warps that
     // hide one another's waits and was slower (2,048 tokens, 8 heads of 64 x 128: 460 -> 570 us)
-    static constexpr int cpt = 1;
+    // In the decayed sum nothing of a token waits for the token before but its own state element, and the walk over
+    // wide keys is bound by the shared-memory reads of k, q and the decays: there two columns a thread win (2,048
+    // tokens, 32 heads of 128 x 128: 640 -> 495 us; at 64 keys they lose, 8 heads of 64 x 128: 163 -> 240 us).
+    static constexpr int cpt = MODE == MODE_DECAYED_SUM && DMAX >= 128 && LANES == 16 ? 2 : 1;
     static constexpr int threads = LANES * (CB / cpt) + (MODE == MODE_GATED_SUM ? 32 : 0);
     static constexpr int resident = LANES == 16 && 768 / threads > 0 ? 768 / threads : 1;
 };
 
 template <int MODE, int DMAX, int CB, int LANES>
-__global__ void __launch_bounds__(StateBlock<MODE, CB, LANES>::threads, StateBlock<MODE, CB, LANES>::resident)
+__global__ void __launch_bounds__(StateBlock<MODE, DMAX, CB, LANES>::threads, StateBlock<MODE, DMAX, CB, LANES>::resident)
 matrix_state_kernel(const MatrixStateArgs p) {
     constexpr int TT = TileTokens<MODE, DMAX, CB>::value;
     constexpr bool DECAYED = MODE == MODE_DECAYED_SUM;
@@ -123,10 +126,10 @@ matrix_state_kernel(const MatrixStateArgs p) {
     constexpr int NG = DMAX / 64;                         // groups of 64 rows
     constexpr int NI = NG * VPT * 4;                      // state rows per thread
     constexpr int CS = CB + 1;                            // columns of o (the last: the normaliser's)
-    constexpr int CPT = StateBlock<MODE, CB, LANES>::cpt;
+    constexpr int CPT = StateBlock<MODE, DMAX, CB, LANES>::cpt;
     constexpr int GROUPS = CB / CPT;                      // threads along the columns
-    constexpr int THREADS = StateBlock<MODE, CB, LANES>::threads;
-    static_assert(DMAX % 64 == 0 && (VPT == 1 || VPT == 4) && THREADS >= 8 * TT && CB % 4 == 0 && CB % CPT == 0, "sizes");
+    constexpr int THREADS = StateBlock<MODE, DMAX, CB, LANES>::threads;
+    static_assert(DMAX % 64 == 0 && (VPT == 1 || VPT == 4) && (DECAYED || THREADS >= 8 * TT) && CB % 4 == 0 && CB % CPT == 0, "sizes");
     __shared__ __align__(16) float ks_[2][TT][DMAX];
     __shared__ __align__(16) float qs_[2][TT][DMAX];
     __shared__ __align__(16) float ds_[DECAYED ? 2 : 1][DECAYED ? TT : 1][DECAYED ? DMAX : 4];
@@ -438,7 +441,7 @@ template <int MODE, int DMAX>
 int launch_cb(const MatrixStateArgs& a, int requests, int cb, int col_blocks, cudaStream_t s) {
     dim3 grid(requests, a.heads, col_blocks);
 #define TI_MS_GO(CB_, LANES_) \
-    matrix_state_kernel<MODE, DMAX, CB_, LANES_><<<grid, StateBlock<MODE, CB_, LANES_>::threads, 0, s>>>(a)
+    matrix_state_kernel<MODE, DMAX, CB_, LANES_><<<grid, StateBlock<MODE, DMAX, CB_, LANES_>::threads, 0, s>>>(a)
     if (a.cut && cb == 8) TI_MS_GO(8, 16);
     else if (a.cut && cb == 16) TI_MS_GO(16, 16);
     else if (a.cut && cb == 32) TI_MS_GO(32, 16);

@@ -475,7 +475,7 @@ class StateOps:
         col_block, o_raw, carry = 0, None, None
         pairs = step.num_requests * heads
         if dv > 128 or (self.cut_state_columns and dv >= 16 and step.max_q_len > 64 and pairs <= 2 * self.num_sms):
-            col_block = 8
+            col_block = 16 if decayed and dk > 64 else 8      # over wide keys a thread walks two columns
             while col_block < 128 and pairs * -(-dv // col_block) > 4 * self.num_sms:
                 col_block *= 2
             o_raw = torch.empty((t, heads * dv), dtype=torch.float32, device=q.device)
