@@ -9,9 +9,10 @@ from .ruvuvik import RuvuvikConfig
 from .feruzen import FeruzenConfig
 from .nekorax import NekoraxConfig
 from .vametar import VametarConfig
+from .saberax import SaberaxConfig
 
 __all__ = [
-    "Architecture", "ConfigError", "FeruzenConfig", "KagoraxConfig", "LayerPlan", "ModelPlan", "NekoraxConfig", "PartSpec", "Qwen3Config", "RuvuvikConfig", "VametarConfig",
+    "Architecture", "ConfigError", "FeruzenConfig", "KagoraxConfig", "LayerPlan", "ModelPlan", "NekoraxConfig", "PartSpec", "Qwen3Config", "RuvuvikConfig", "SaberaxConfig", "VametarConfig",
     "ScheduleEntry", "architecture_of", "default_schedule", "get_architecture",
     "known_architectures", "load_config", "read_config_json", "register_architecture",
 ]

@@ -12,7 +12,8 @@
 //
 // Epilogues: store, accumulate into C (the residual stream; optionally through a gate, C += scale
 // sigmoid(gate + bias) * sum), or SwiGLU: W holds, in every strip,
-// 8 gate rows followed by their 8 up rows, and out[m, j] = silu(gate_j) * up_j in bfloat16.
+// 8 gate rows followed by their 8 up rows, and out[m, j] = silu(gate_j) * up_j in bfloat16; or an activation of
+// one value per output.
 #include "common.cuh"
 #include "glu.cuh"
 
@@ -22,7 +23,7 @@ constexpr int WARPS = 8;
 constexpr int STRIP = 16;
 constexpr int CHUNK = 32;
 
-enum { MODE_STORE = 0, MODE_ACCUMULATE = 1, MODE_SWIGLU = 2, MODE_XIELU = 3 };
+enum { MODE_STORE = 0, MODE_ACCUMULATE = 1, MODE_SWIGLU = 2, MODE_XIELU = 3, MODE_UNARY = 4 };
 
 __device__ __forceinline__ uint4 ld_stream(const void* p) {
     uint4 v;
@@ -39,10 +40,10 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], unsigned a0, unsigned a1
                  : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
 
-// A second product over the same number of rows and the same k in the same launch: the blocks from `first_block` on
-// (0: there is none) store its strips.  Two products of a decode step that depend on nothing of each other (a
+// A second product over the same number of rows (with a k of its own) in the same launch: the blocks from `first_block`
+// on (0: there is none) store its strips.  Two products of a decode step that depend on nothing of each other (a
 // sublayer's first product and its gate) then wait for the kernel before them once.
-struct SecondProduct { const bf16* a; const bf16* w; float* c; int n, lda, ldw, ldc; unsigned first_block; };
+struct SecondProduct { const bf16* a; const bf16* w; float* c; int n, k, lda, ldw, ldc; unsigned first_block; };
 
 // ROWS = 16: a block owns 16 rows of W.  ROWS = 8: it owns 8 (the upper half of the MMA's A
 // operand is zero), which doubles the number of blocks for narrow outputs.
@@ -66,7 +67,7 @@ gemm_skinny_kernel(const bf16* a, const bf16* __restrict__ w, float* __restrict_
     if (second.first_block > 0 && blockIdx.x >= second.first_block) {      // the blocks of the second product
         n0 = (blockIdx.x - second.first_block) * ROWS;
         a = second.a; w = second.w; c = second.c;
-        n = second.n; lda = second.lda; ldw = second.ldw; ldc = second.ldc;
+        n = second.n; k = second.k; lda = second.lda; ldw = second.ldw; ldc = second.ldc;
         mode = MODE_STORE;
     }
     // rows past N are read from the last row and never stored
@@ -185,7 +186,9 @@ gemm_skinny_kernel(const bf16* a, const bf16* __restrict__ w, float* __restrict_
             float sum = 0.0f;
 #pragma unroll
             for (int wp = 0; wp < WARPS; ++wp) sum += part[wp][i][tok];
-            if (mode == MODE_XIELU) {          // act_p z^2 + z/2 above zero, act_q (exp(z) - 1 - z) + z/2 below
+            if (mode == MODE_UNARY) {
+                if (n0 + i < n) out_act[(size_t)tok * ld_act + n0 + i] = __float2bfloat16_rn(unary_activation(glu_kind, sum));
+            } else if (mode == MODE_XIELU) {          // act_p z^2 + z/2 above zero, act_q (exp(z) - 1 - z) + z/2 below
                 const float y = sum > 0.0f ? fmaf(act_p * sum, sum, 0.5f * sum) : fmaf(act_q, expm1f(sum) - sum, 0.5f * sum);
                 if (n0 + i < n) out_act[(size_t)tok * ld_act + n0 + i] = __float2bfloat16_rn(y);
             } else if (n0 + i < n) {
@@ -205,8 +208,8 @@ extern "C" int ti_gemm_skinny_supported(int m, int n, int k, int lda, int ldw) {
 // 3: out_act[m, n] = xielu(a w^T) with the activation's two factors.
 static int skinny(const void* a, const void* w, float* c, void* out_act, int m, int n, int k, int lda, int ldw,
                   int ldc, int ld_act, int mode, int glu_kind, float act_p, float act_q, void* stream,
-                  AddGate add = AddGate{nullptr, 0, nullptr, 0.0f},
-                  SecondProduct second = SecondProduct{nullptr, nullptr, nullptr, 0, 0, 0, 0, 0}) {
+                  AddGate add = AddGate{nullptr, 0, nullptr, 1.0f},
+                  SecondProduct second = SecondProduct{nullptr, nullptr, nullptr, 0, 0, 0, 0, 0, 0}) {
     if (m == 0 || n == 0) return 0;
     TI_REQUIRE(ti_gemm_skinny_supported(m, n, k, lda, ldw),
                "gemm_skinny: M=%d (1..64), K=%d (multiple of 32) or row strides %d, %d (multiples of 8) "
@@ -219,6 +222,7 @@ static int skinny(const void* a, const void* w, float* c, void* out_act, int m, 
     const bool narrow = mode != MODE_SWIGLU && (n + STRIP - 1) / STRIP + (second.n + STRIP - 1) / STRIP < 128;
     const int rows = narrow ? 8 : STRIP;
     unsigned blocks = (unsigned)((n + rows - 1) / rows);
+    const int longest = k > second.k ? k : second.k;
     if (second.n > 0) {
         second.first_block = blocks;
         blocks += (unsigned)((second.n + rows - 1) / rows);
@@ -228,11 +232,11 @@ static int skinny(const void* a, const void* w, float* c, void* out_act, int m, 
         ti_launch_pdl(gemm_skinny_kernel<NT, 8, 8>, blocks, WARPS * 32, 0, s,      \
                       (const bf16*)a, (const bf16*)w, c, (bf16*)out_act, m, n, k, lda, ldw, ldc,    \
                       ld_act, mode, glu_kind, act_p, act_q, add, second);                                                                \
-    else if (k <= SHORT_K && mode == MODE_STORE && NT <= 2)                                         \
+    else if (longest <= SHORT_K && mode == MODE_STORE && NT <= 2)                                         \
         ti_launch_pdl((gemm_skinny_kernel<NT <= 2 ? NT : 1, 16, 4, true>), blocks, \
                       WARPS * 32, 0, s, (const bf16*)a, (const bf16*)w, c, (bf16*)out_act, m, n, k, \
                       lda, ldw, ldc, ld_act, mode, glu_kind, act_p, act_q, add, second);                                   \
-    else if (k <= SHORT_K)                                                                          \
+    else if (longest <= SHORT_K)                                                                          \
         ti_launch_pdl(gemm_skinny_kernel<NT, 16, 4>, blocks,                                        \
                       WARPS * 32, 0, s, (const bf16*)a, (const bf16*)w, c, (bf16*)out_act, m, n, k, \
                       lda, ldw, ldc, ld_act, mode, glu_kind, act_p, act_q, add, second);                                   \
@@ -262,32 +266,40 @@ extern "C" int ti_gemm_skinny_glu(const void* a, const void* w, void* out_act, i
     return skinny(a, w, nullptr, out_act, m, n, k, lda, ldw, 0, ld_act, MODE_SWIGLU, glu_kind, glu_limit, glu_alpha, stream);
 }
 
-// c += scale sigmoid(gate + bias) * (a w^T), element by element; gate float32 [m, n] (row stride ld_gate), bias [n]
+// c += scale sigmoid(gate + bias) * (a w^T), element by element; gate float32 [m, n] (row stride ld_gate), bias [n];
+// without a gate c += scale * (a w^T)
 extern "C" int ti_gemm_skinny_gated(const void* a, const void* w, float* c, int m, int n, int k, int lda, int ldw,
                                     int ldc, const float* gate, int ld_gate, const float* bias, float scale,
                                     void* stream) {
-    TI_REQUIRE(gate != nullptr && bias != nullptr, "gemm_skinny_gated: a gate and its bias");
+    TI_REQUIRE((gate != nullptr) == (bias != nullptr), "gemm_skinny_gated: a gate and its bias");
     return skinny(a, w, c, nullptr, m, n, k, lda, ldw, ldc, 0, MODE_ACCUMULATE, GLU_SILU, 0.0f, 0.0f, stream,
                   AddGate{gate, ld_gate, bias, scale});
 }
 
-// Two products of m rows and the same k in one launch: the first stores its float32 rows into c, or (glu_kind >= 0)
+// Two products of m rows in one launch: the first stores its float32 rows into c, or (glu_kind >= 0)
 // its gated activation over strips of 8 and 8 into out_act; the second stores a2 w2^T into c2.
 extern "C" int ti_gemm_skinny_pair(const void* a, const void* w, float* c, void* out_act, int m, int n, int k, int lda,
                                    int ldw, int ldc, int ld_act, int glu_kind, float glu_limit, float glu_alpha,
-                                   const void* a2, const void* w2, float* c2, int n2, int lda2, int ldw2, int ldc2,
+                                   const void* a2, const void* w2, float* c2, int n2, int k2, int lda2, int ldw2, int ldc2,
                                    void* stream) {
     if (m == 0 || n == 0 || n2 == 0) return 0;
     TI_REQUIRE(glu_kind <= GLU_GELU_TANH, "gemm_skinny_pair: activation %d", glu_kind);
-    TI_REQUIRE(ti_gemm_skinny_supported(m, n2, k, lda2, ldw2) && (uintptr_t)a2 % 16 == 0 && (uintptr_t)w2 % 16 == 0,
+    TI_REQUIRE(ti_gemm_skinny_supported(m, n2, k2, lda2, ldw2) && (uintptr_t)a2 % 16 == 0 && (uintptr_t)w2 % 16 == 0,
                "gemm_skinny_pair: the second product's operands");
     return skinny(a, w, c, out_act, m, n, k, lda, ldw, ldc, ld_act, glu_kind < 0 ? MODE_STORE : MODE_SWIGLU,
-                  glu_kind < 0 ? GLU_SILU : glu_kind, glu_limit, glu_alpha, stream, AddGate{nullptr, 0, nullptr, 0.0f},
-                  SecondProduct{(const bf16*)a2, (const bf16*)w2, c2, n2, lda2, ldw2, ldc2, 0});
+                  glu_kind < 0 ? GLU_SILU : glu_kind, glu_limit, glu_alpha, stream, AddGate{nullptr, 0, nullptr, 1.0f},
+                  SecondProduct{(const bf16*)a2, (const bf16*)w2, c2, n2, k2, lda2, ldw2, ldc2, 0});
 }
 
 // out_act[m, n] (bfloat16) = xielu(a w^T): act_p z^2 + z/2 for z > 0, act_q (exp(z) - 1 - z) + z/2 otherwise
 extern "C" int ti_gemm_skinny_xielu(const void* a, const void* w, void* out_act, int m, int n, int k, int lda,
                                     int ldw, int ld_act, float act_p, float act_q, void* stream) {
     return skinny(a, w, nullptr, out_act, m, n, k, lda, ldw, 0, ld_act, MODE_XIELU, GLU_SILU, act_p, act_q, stream);
+}
+
+// out_act[m, n] (bfloat16) = act(a w^T) with the activation of one value `act` of glu.cuh
+extern "C" int ti_gemm_skinny_unary(const void* a, const void* w, void* out_act, int m, int n, int k, int lda,
+                                    int ldw, int ld_act, int act, void* stream) {
+    TI_REQUIRE(act == ACT_RELU2, "gemm_skinny_unary: activation %d", act);
+    return skinny(a, w, nullptr, out_act, m, n, k, lda, ldw, 0, ld_act, MODE_UNARY, act, 0.0f, 0.0f, stream);
 }

@@ -11,7 +11,8 @@
 // warps 2-9 read a finished accumulator with tcgen05.ld (a warp reads the 32 TMEM lanes = rows
 // that its position in the warpgroup allows) and run the epilogue while the next tile's
 // products already fill the other accumulator.  Epilogues: store, accumulate into C (the
-// residual stream; optionally through a gate, C += scale sigmoid(gate + bias) * sum), SwiGLU over 8 gate + 8 up columns into bfloat16, or (BN = 256) the QKV
+// residual stream; optionally through a gate, C += scale sigmoid(gate + bias) * sum), SwiGLU over 8 gate + 8 up columns
+// into bfloat16, an activation of one value per column into bfloat16, or (BN = 256) the QKV
 // epilogue of qkv_epilogue.cuh: head norm, rotation and the store into the paged cache.  Rows and columns past
 // M, N and K are zero-filled by TMA on the way in and skipped on the way out.
 //
@@ -39,7 +40,7 @@ template <int BN> struct Tile {
     static constexpr unsigned TMEM_COLS = 2 * BN;     // two accumulators
 };
 
-enum { MODE_STORE = 0, MODE_ACCUMULATE = 1, MODE_SWIGLU = 2, MODE_QKV = 3 };
+enum { MODE_STORE = 0, MODE_ACCUMULATE = 1, MODE_SWIGLU = 2, MODE_QKV = 3, MODE_UNARY = 4 };
 enum { TI_ERR_TIMEOUT = 2 };
 
 // Work unit `unit` of a product whose K is cut into `splits` runs: its tile and its k blocks.
@@ -244,6 +245,20 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                         *reinterpret_cast<uint4*>(out_act + (size_t)row * ld_act + (col + half * 16) / 2) =
                             make_uint4(packed[0], packed[1], packed[2], packed[3]);
                     }
+                } else if (mode == MODE_UNARY) {
+#pragma unroll
+                    for (int i = 0; i < 32; i += 8) {
+                        if (col + i >= n) break;
+                        unsigned packed[4];
+#pragma unroll
+                        for (int j = 0; j < 4; ++j) {
+                            __nv_bfloat162 y = __floats2bfloat162_rn(unary_activation(glu.kind, v[i + 2 * j]),
+                                                                     unary_activation(glu.kind, v[i + 2 * j + 1]));
+                            packed[j] = *reinterpret_cast<unsigned*>(&y);
+                        }
+                        *reinterpret_cast<uint4*>(out_act + (size_t)row * ld_act + col + i) =
+                            make_uint4(packed[0], packed[1], packed[2], packed[3]);
+                    }
                 } else {
                     float* dst = c + (size_t)row * ldc + col;
                     // whole 32-byte sectors where the rows allow it: a thread's stores are a row each
@@ -355,7 +370,7 @@ int choose_splits(int m, int n, int k, int mode, int sms) {
 int launch_tiles(const void* a, const void* w, const qkv::Epilogue& e, float* c, void* out_act, int m, int n,
                  int k, int lda, int ldw, int ldc, int ld_act, int mode, int width, float* ws, int splits,
                  int* status, void* stream, bool add_runs = true, GluArgs glu = GluArgs{GLU_SILU, 0.0f, 0.0f},
-                 AddGate add = AddGate{nullptr, 0, nullptr, 0.0f}) {
+                 AddGate add = AddGate{nullptr, 0, nullptr, 1.0f}) {
     int device = 0, sms = 0;
     cudaGetDevice(&device);
     cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, device);
@@ -407,6 +422,7 @@ int launch_tiles(const void* a, const void* w, const qkv::Epilogue& e, float* c,
 extern "C" int ti_gemm_tcgen05_supported(int m, int n, int k, int lda, int ldw, int ldc, int mode) {
     if (m < 1 || n < 1 || k < 8 || k % 8 || lda % 8 || ldw % 8) return 0;
     if (mode == MODE_SWIGLU) return n % 16 == 0;
+    if (mode == MODE_UNARY) return n % 8 == 0;
     return n % 4 == 0 && ldc % 4 == 0;
 }
 
@@ -427,7 +443,7 @@ extern "C" int ti_gemm_tcgen05_add_runs(const float* ws, float* c, int m, int n,
                "gemm_tcgen05_add_runs: N=%d and the row stride %d must be multiples of 4", n, ldc);
     const long long quads = (long long)m * (n / 4);
     ti_launch_pdl(gemm_split_merge_kernel, (unsigned)((quads + 255) / 256), 256, 0, (cudaStream_t)stream, ws, c, m,
-                  n, ldc, runs, accumulate ? 1 : 0, AddGate{nullptr, 0, nullptr, 0.0f});
+                  n, ldc, runs, accumulate ? 1 : 0, AddGate{nullptr, 0, nullptr, 1.0f});
     return ti_check_launch("gemm_split_merge");
 }
 
@@ -467,15 +483,15 @@ extern "C" int ti_gemm_tcgen05(const void* a, const void* w, float* c, void* out
                                int k, int lda, int ldw, int ldc, int ld_act, int mode, float* ws,
                                int leave_runs, int* status, void* stream) {
     return gemm_tcgen05(a, w, c, out_act, m, n, k, lda, ldw, ldc, ld_act, mode, ws, leave_runs, status, stream,
-                        AddGate{nullptr, 0, nullptr, 0.0f});
+                        AddGate{nullptr, 0, nullptr, 1.0f});
 }
 
 // c += scale sigmoid(gate + bias) * (a w^T), element by element; gate float32 [m, n] (row stride ld_gate), bias [n],
-// both on 16 bytes; the runs of a cut K pass the gate in the launch that adds them
+// both on 16 bytes; without a gate c += scale * (a w^T); the runs of a cut K pass the gate in the launch that adds them
 extern "C" int ti_gemm_tcgen05_gated(const void* a, const void* w, float* c, int m, int n, int k, int lda, int ldw,
                                      int ldc, float* ws, const float* gate, int ld_gate, const float* bias, float scale,
                                      int* status, void* stream) {
-    TI_REQUIRE((uintptr_t)gate % 16 == 0 && (uintptr_t)bias % 16 == 0 && ld_gate % 4 == 0 && gate != nullptr && bias != nullptr,
+    TI_REQUIRE((uintptr_t)gate % 16 == 0 && (uintptr_t)bias % 16 == 0 && ld_gate % 4 == 0 && (gate != nullptr) == (bias != nullptr),
                "gemm_tcgen05_gated: the gate's rows and the bias must start on 16 bytes");
     return gemm_tcgen05(a, w, c, nullptr, m, n, k, lda, ldw, ldc, 0, MODE_ACCUMULATE, ws, 0, status, stream,
                         AddGate{gate, ld_gate, bias, scale});
@@ -483,19 +499,19 @@ extern "C" int ti_gemm_tcgen05_gated(const void* a, const void* w, float* c, int
 
 // Grouped product: row tile i (128 rows of a) is multiplied by the i-th named group's weights,
 // w + group_of_tile[i] * n * ldw; `tiles_m_dev` (device) says how many row tiles there are, at most
-// m_max / 128.  c (MODE_STORE) or out_act (MODE_SWIGLU) has m_max rows.  Not a dependent launch.
+// m_max / 128.  c (MODE_STORE) or out_act (MODE_SWIGLU, MODE_UNARY) has m_max rows.  Not a dependent launch.
 static int gemm_tcgen05_grouped_impl(const void* a, const void* w, float* c, void* out_act, int m_max, int n,
                                      int k, int lda, int ldw, int ldc, int ld_act, int mode, int groups,
                                      const int* group_of_tile, const int* tiles_m_dev, int* status,
                                      void* stream, GluArgs glu) {
     if (m_max == 0 || n == 0) return 0;
-    TI_REQUIRE(mode == MODE_STORE || mode == MODE_SWIGLU, "gemm_tcgen05_grouped: mode %d", mode);
+    TI_REQUIRE(mode == MODE_STORE || mode == MODE_SWIGLU || mode == MODE_UNARY, "gemm_tcgen05_grouped: mode %d", mode);
     TI_REQUIRE(m_max % BM == 0 && ti_gemm_tcgen05_supported(m_max, n, k, lda, ldw, ldc, mode),
                "gemm_tcgen05_grouped: rows %d must be a multiple of %d, K=%d and the row strides multiples "
                "of 8, N=%d a multiple of 4 (16 with SwiGLU)", m_max, BM, k, n);
     TI_REQUIRE((uintptr_t)a % 16 == 0 && (uintptr_t)w % 16 == 0 && group_of_tile != nullptr && tiles_m_dev != nullptr,
                "gemm_tcgen05_grouped: operands must be 16-byte aligned and the tile list given");
-    TI_REQUIRE(mode == MODE_SWIGLU ? ((uintptr_t)out_act % 16 == 0 && ld_act % 8 == 0) : (uintptr_t)c % 16 == 0,
+    TI_REQUIRE(mode != MODE_STORE ? ((uintptr_t)out_act % 16 == 0 && ld_act % 8 == 0) : (uintptr_t)c % 16 == 0,
                "gemm_tcgen05_grouped: the output must be 16-byte aligned");
     int device = 0, sms = 0;
     cudaGetDevice(&device);
@@ -520,11 +536,11 @@ static int gemm_tcgen05_grouped_impl(const void* a, const void* w, float* c, voi
     if (width == 256)
         gemm_tcgen05_kernel<256><<<grid, THREADS, Tile<256>::SMEM, (cudaStream_t)stream>>>(
             map_a, map_w, qkv::Epilogue{}, c, (bf16*)out_act, m_max, n, k, ldc, ld_act, mode, nullptr, 1, status,
-            group_of_tile, tiles_m_dev, glu, AddGate{nullptr, 0, nullptr, 0.0f});
+            group_of_tile, tiles_m_dev, glu, AddGate{nullptr, 0, nullptr, 1.0f});
     else
         gemm_tcgen05_kernel<128><<<grid, THREADS, Tile<128>::SMEM, (cudaStream_t)stream>>>(
             map_a, map_w, qkv::Epilogue{}, c, (bf16*)out_act, m_max, n, k, ldc, ld_act, mode, nullptr, 1, status,
-            group_of_tile, tiles_m_dev, glu, AddGate{nullptr, 0, nullptr, 0.0f});
+            group_of_tile, tiles_m_dev, glu, AddGate{nullptr, 0, nullptr, 1.0f});
     return ti_check_launch("gemm_tcgen05_grouped");
 }
 
@@ -537,26 +553,31 @@ extern "C" int ti_gemm_tcgen05_grouped(const void* a, const void* w, float* c, v
 }
 
 // The grouped product whose epilogue is the gated activation `glu_kind` of glu.cuh over groups of
-// 8 gate + 8 up columns: out_act[m_max, n/2].
+// 8 gate + 8 up columns, out_act[m_max, n/2], or an activation of one value, out_act[m_max, n].
 extern "C" int ti_gemm_tcgen05_grouped_glu(const void* a, const void* w, void* out_act, int m_max, int n, int k,
                                            int lda, int ldw, int ld_act, int groups, const int* group_of_tile,
                                            const int* tiles_m_dev, int glu_kind, float glu_limit, float glu_alpha,
                                            int* status, void* stream) {
-    TI_REQUIRE(glu_kind >= GLU_SILU && glu_kind <= GLU_GELU_TANH, "gemm_tcgen05_grouped_glu: activation %d", glu_kind);
-    return gemm_tcgen05_grouped_impl(a, w, nullptr, out_act, m_max, n, k, lda, ldw, 0, ld_act, MODE_SWIGLU, groups,
+    TI_REQUIRE((glu_kind >= GLU_SILU && glu_kind <= GLU_GELU_TANH) || glu_kind == ACT_RELU2,
+               "gemm_tcgen05_grouped_glu: activation %d", glu_kind);
+    return gemm_tcgen05_grouped_impl(a, w, nullptr, out_act, m_max, n, k, lda, ldw, 0, ld_act,
+                                     act_is_gated(glu_kind) ? MODE_SWIGLU : MODE_UNARY, groups,
                                      group_of_tile, tiles_m_dev, status, stream, GluArgs{glu_kind, glu_limit, glu_alpha});
 }
 
 // out_act[m, n/2] = act(gate, up) of a w^T over groups of 8 gate + 8 up columns, with the gated
-// activation `glu_kind` of glu.cuh in the epilogue (K uncut).
+// activation `glu_kind` of glu.cuh in the epilogue (K uncut), or out_act[m, n] = act(a w^T) with an
+// activation of one value.
 extern "C" int ti_gemm_tcgen05_glu(const void* a, const void* w, void* out_act, int m, int n, int k, int lda,
                                    int ldw, int ld_act, int glu_kind, float glu_limit, float glu_alpha, int* status,
                                    void* stream) {
     if (m == 0 || n == 0) return 0;
-    TI_REQUIRE(glu_kind >= GLU_SILU && glu_kind <= GLU_GELU_TANH, "gemm_tcgen05_glu: activation %d", glu_kind);
-    TI_REQUIRE(ti_gemm_tcgen05_supported(m, n, k, lda, ldw, 0, MODE_SWIGLU),
-               "gemm_tcgen05_glu: K=%d and the row strides %d, %d must be multiples of 8, N=%d a multiple of 16", k, lda,
-               ldw, n);
+    TI_REQUIRE((glu_kind >= GLU_SILU && glu_kind <= GLU_GELU_TANH) || glu_kind == ACT_RELU2,
+               "gemm_tcgen05_glu: activation %d", glu_kind);
+    const int mode = act_is_gated(glu_kind) ? MODE_SWIGLU : MODE_UNARY;
+    TI_REQUIRE(ti_gemm_tcgen05_supported(m, n, k, lda, ldw, 0, mode),
+               "gemm_tcgen05_glu: K=%d and the row strides %d, %d must be multiples of 8, N=%d a multiple of 16 (8 without "
+               "a gate)", k, lda, ldw, n);
     TI_REQUIRE((uintptr_t)a % 16 == 0 && (uintptr_t)w % 16 == 0 && (uintptr_t)out_act % 16 == 0 && ld_act % 8 == 0,
                "gemm_tcgen05_glu: operands and output must be 16-byte aligned");
     int device = 0, sms = 0;
@@ -564,7 +585,7 @@ extern "C" int ti_gemm_tcgen05_glu(const void* a, const void* w, void* out_act, 
     cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, device);
     const int tiles_m = (m + BM - 1) / BM;
     const int width = tiles_m * ((n + 255) / 256) >= sms ? 256 : tiles_m * ((n + 127) / 128) * 2 >= sms ? 128 : 64;
-    return launch_tiles(a, w, qkv::Epilogue{}, nullptr, out_act, m, n, k, lda, ldw, 0, ld_act, MODE_SWIGLU, width,
+    return launch_tiles(a, w, qkv::Epilogue{}, nullptr, out_act, m, n, k, lda, ldw, 0, ld_act, mode, width,
                         nullptr, 1, status, stream, true, GluArgs{glu_kind, glu_limit, glu_alpha});
 }
 

@@ -280,7 +280,7 @@ namespace {
 
 int launch_pairs(const void* a, const void* w, const qkv::Epilogue& e, float* c, void* out_act, int m, int n,
                  int k, int lda, int ldw, int ldc, int ld_act, int mode, int* status, void* stream,
-                 AddGate add = AddGate{nullptr, 0, nullptr, 0.0f}) {
+                 AddGate add = AddGate{nullptr, 0, nullptr, 1.0f}) {
     int device = 0, sms = 0;
     cudaGetDevice(&device);
     cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, device);
@@ -319,7 +319,7 @@ extern "C" int ti_gemm_tcgen05_2sm(const void* a, const void* w, float* c, void*
     return launch_pairs(a, w, qkv::Epilogue{}, c, out_act, m, n, k, lda, ldw, ldc, ld_act, mode, status, stream);
 }
 
-// c += scale sigmoid(gate + bias) * (a w^T): as ti_gemm_tcgen05_gated, K never cut
+// c += scale sigmoid(gate + bias) * (a w^T), or without a gate c += scale * (a w^T): as ti_gemm_tcgen05_gated, K never cut
 extern "C" int ti_gemm_tcgen05_2sm_gated(const void* a, const void* w, float* c, int m, int n, int k, int lda, int ldw,
                                          int ldc, const float* gate, int ld_gate, const float* bias, float scale,
                                          int* status, void* stream) {
@@ -328,7 +328,7 @@ extern "C" int ti_gemm_tcgen05_2sm_gated(const void* a, const void* w, float* c,
                "gemm_tcgen05_2sm_gated: K=%d and the row strides %d, %d must be multiples of 8, N=%d a multiple of 4", k, lda,
                ldw, n);
     TI_REQUIRE((uintptr_t)a % 16 == 0 && (uintptr_t)w % 16 == 0 && (uintptr_t)c % 16 == 0 && (uintptr_t)gate % 16 == 0 &&
-               (uintptr_t)bias % 16 == 0 && ld_gate % 4 == 0 && gate != nullptr && bias != nullptr,
+               (uintptr_t)bias % 16 == 0 && ld_gate % 4 == 0 && (gate != nullptr) == (bias != nullptr),
                "gemm_tcgen05_2sm_gated: operands, output, the gate's rows and the bias must start on 16 bytes");
     return launch_pairs(a, w, qkv::Epilogue{}, c, nullptr, m, n, k, lda, ldw, ldc, 0, MODE_ACCUMULATE, status, stream,
                         AddGate{gate, ld_gate, bias, scale});

@@ -358,14 +358,15 @@ extern "C" int ti_gemm_tcgen05_few(const void* a, const void* w, float* c, void*
                                    int ldw, int ldc, int ld_act, int mode, float* ws, int* tickets, int* status,
                                    void* stream) {
     return few(a, w, c, out_act, m, n, k, lda, ldw, ldc, ld_act, mode, ws, tickets, status, stream,
-               AddGate{nullptr, 0, nullptr, 0.0f});
+               AddGate{nullptr, 0, nullptr, 1.0f});
 }
 
-// c += scale sigmoid(gate + bias) * (a w^T), element by element; gate float32 [m, n] (row stride ld_gate), bias [n]
+// c += scale sigmoid(gate + bias) * (a w^T), element by element; gate float32 [m, n] (row stride ld_gate), bias [n];
+// without a gate c += scale * (a w^T)
 extern "C" int ti_gemm_tcgen05_few_gated(const void* a, const void* w, float* c, int m, int n, int k, int lda, int ldw,
                                          int ldc, float* ws, int* tickets, const float* gate, int ld_gate,
                                          const float* bias, float scale, int* status, void* stream) {
-    TI_REQUIRE(gate != nullptr && bias != nullptr, "gemm_tcgen05_few_gated: a gate and its bias");
+    TI_REQUIRE((gate != nullptr) == (bias != nullptr), "gemm_tcgen05_few_gated: a gate and its bias");
     return few(a, w, c, nullptr, m, n, k, lda, ldw, ldc, 0, MODE_ACCUMULATE, ws, tickets, status, stream,
                AddGate{gate, ld_gate, bias, scale});
 }

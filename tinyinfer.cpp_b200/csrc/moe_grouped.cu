@@ -7,8 +7,10 @@
 //  2. moe_grouped<GATED>: a block takes one tile of rows and 64 output columns of its expert:
 //     rows of h gathered by token, the expert's gate and up rows, float32 accumulation, and
 //     y = silu(w g) * (w u) in the epilogue (w: the pair's weight), stored in sorted order; with
-//     another activation (glu.cuh) the weight scales the output instead: y = w act(g, u).
-//  3. moe_grouped<!GATED>: the same walk over y and the expert's down rows, 128 output columns a
+//     another activation (glu.cuh) the weight scales the output instead: y = w act(g, u).  With an
+//     activation of one value (moe_grouped<UNARY>) an expert has up rows only, y = w act(u), 128
+//     output columns a block.
+//  3. moe_grouped<DOWN>: the same walk over y and the expert's down rows, 128 output columns a
 //     block; the float32 result goes to the pair's own row of a scratch.
 //  4. moe_combine: residual[t] += the rows of t's pairs, in slot order.
 //
@@ -111,7 +113,9 @@ moe_sort_kernel(const int* __restrict__ ids, int n_pairs, int experts, int* __re
     }
 }
 
-template <bool GATED>
+enum { KIND_DOWN = 0, KIND_GATED = 1, KIND_UNARY = 2 };
+
+template <int KIND>
 __global__ void __launch_bounds__(THREADS)
 moe_grouped_kernel(const bf16* a, int lda, const int* __restrict__ sorted_slot,
                    const int* __restrict__ tiles, const int* __restrict__ meta, int top,
@@ -123,6 +127,7 @@ moe_grouped_kernel(const bf16* a, int lda, const int* __restrict__ sorted_slot,
     const int tile = blockIdx.y;
     if (tile >= meta[0]) return;
     const int expert = tiles[tile * 3], row0 = tiles[tile * 3 + 1], rows = tiles[tile * 3 + 2];
+    constexpr bool GATED = KIND == KIND_GATED;
     constexpr int BN_OUT = GATED ? BNW / 2 : BNW;       // output columns of a block
     const int n0 = blockIdx.x * BN_OUT;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -132,7 +137,7 @@ moe_grouped_kernel(const bf16* a, int lda, const int* __restrict__ sorted_slot,
     if (threadIdx.x < BM) {
         const int r = threadIdx.x;
         int src = -1;
-        if (r < rows) src = GATED ? sorted_slot[row0 + r] / top : row0 + r;
+        if (r < rows) src = KIND != KIND_DOWN ? sorted_slot[row0 + r] / top : row0 + r;
         row_src[r] = src;
     }
     __syncthreads();
@@ -234,6 +239,17 @@ moe_grouped_kernel(const bf16* a, int lda, const int* __restrict__ sorted_slot,
                         y1 = w * glu_activation(act, acc[i][j][2 * half + 1], acc[i][j + 4][2 * half + 1], act_limit, act_alpha);
                     }
                     *reinterpret_cast<__nv_bfloat162*>(dst + col) = __floats2bfloat162_rn(y0, y1);
+                }
+            } else if (KIND == KIND_UNARY) {
+                const float w = weights[sorted_slot[row0 + r]];
+                bf16* dst = y_sorted + (size_t)(row0 + r) * n;
+#pragma unroll
+                for (int j = 0; j < 8; ++j) {
+                    const int col = n0 + wn * 64 + j * 8 + tq * 2;
+                    if (col >= n) continue;
+                    *reinterpret_cast<__nv_bfloat162*>(dst + col) =
+                        __floats2bfloat162_rn(w * unary_activation(act, acc[i][j][2 * half]),
+                                              w * unary_activation(act, acc[i][j][2 * half + 1]));
                 }
             } else {
                 float* dst = out_rows + (size_t)sorted_slot[row0 + r] * n;
@@ -418,17 +434,24 @@ extern "C" int ti_moe_grouped(const void* h, int h_stride, const void* w_gate_up
     constexpr int SMEM = STAGES * STAGE_BYTES;
     static TiPerDevice configured;
     if (configured.first_use()) {
-        cudaError_t e1 = cudaFuncSetAttribute(moe_grouped_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
-        cudaError_t e2 = cudaFuncSetAttribute(moe_grouped_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
-        if (e1 != cudaSuccess || e2 != cudaSuccess) return ti_fail("moe_grouped: cannot set the shared memory size");
+        cudaError_t e1 = cudaFuncSetAttribute(moe_grouped_kernel<KIND_GATED>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
+        cudaError_t e2 = cudaFuncSetAttribute(moe_grouped_kernel<KIND_DOWN>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
+        cudaError_t e3 = cudaFuncSetAttribute(moe_grouped_kernel<KIND_UNARY>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
+        if (e1 != cudaSuccess || e2 != cudaSuccess || e3 != cudaSuccess) return ti_fail("moe_grouped: cannot set the shared memory size");
         configured.mark();
     }
-    dim3 g1((ff + BNW / 2 - 1) / (BNW / 2), max_tiles);
-    moe_grouped_kernel<true><<<g1, THREADS, SMEM, s>>>(
-        (const bf16*)h, h_stride, sorted_slot, tiles, meta, top, (const bf16*)w_gate_up, interleaved, ff, width,
-        weights, (bf16*)y_sorted, nullptr, act, act_limit, act_alpha);
+    const int cols = act_is_gated(act) ? BNW / 2 : BNW;
+    dim3 g1((ff + cols - 1) / cols, max_tiles);
+    if (act_is_gated(act))
+        moe_grouped_kernel<KIND_GATED><<<g1, THREADS, SMEM, s>>>(
+            (const bf16*)h, h_stride, sorted_slot, tiles, meta, top, (const bf16*)w_gate_up, interleaved, ff, width,
+            weights, (bf16*)y_sorted, nullptr, act, act_limit, act_alpha);
+    else
+        moe_grouped_kernel<KIND_UNARY><<<g1, THREADS, SMEM, s>>>(
+            (const bf16*)h, h_stride, sorted_slot, tiles, meta, top, (const bf16*)w_gate_up, 0, ff, width,
+            weights, (bf16*)y_sorted, nullptr, act, act_limit, act_alpha);
     dim3 g2((width + BNW - 1) / BNW, max_tiles);
-    moe_grouped_kernel<false><<<g2, THREADS, SMEM, s>>>(
+    moe_grouped_kernel<KIND_DOWN><<<g2, THREADS, SMEM, s>>>(
         (const bf16*)y_sorted, ff, sorted_slot, tiles, meta, top, (const bf16*)w_down, 0, width, ff,
         nullptr, nullptr, out_rows, 0, 0.0f, 0.0f);
     const size_t total = (size_t)num_tokens * width;

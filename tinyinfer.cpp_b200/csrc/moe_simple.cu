@@ -5,10 +5,10 @@
 //    sigmoid of their logits as weights (or, `softmax`, their share of the softmax over all
 //    experts, not renormalised); one more column of the same product, if there is one,
 //    becomes the sigmoid gate of a shared expert.
-//  * router_choose: scores s = softmax over all outputs of the router; the choice looks at s + correction,
-//    only inside the `keep` groups (of `groups` equal runs of neighbours) whose largest such value is
-//    largest, and takes the `top` largest there (ties: the lower index); the weights are the chosen
-//    outputs' s, as they are.
+//  * router_choose: scores s = softmax over all outputs of the router, or the sigmoid of each; the choice looks
+//    at s + correction, only inside the `keep` groups (of `groups` equal runs of neighbours) whose largest such
+//    value, or sum of the two largest, is largest, and takes the `top` largest there (ties: the lower index);
+//    the weights are the chosen outputs' s, as they are or divided by their sum, times a factor.
 //  An index at or behind the number of stacked experts names an *identity expert*: it has no tensors, and
 //  its output is the token's input times the weight.  The kernels below skip its products and add
 //  `w h[t]` where the slots are summed.
@@ -16,10 +16,12 @@
 //    the expert and weight of the token's slot s (an expert's gate and up rows are stacked in one
 //    matrix, interleaved in strips of 8 or one after the other).  The weight stands for a scaling of the
 //    expert's input: (Wgate (w h), Wup (w h)) = (w g, w u).  With another activation (glu.cuh) the
-//    weight scales the expert's output: y = w act(g, u).
+//    weight scales the expert's output: y = w act(g, u).  With an activation of one value an expert has no
+//    gate rows: y = w act(u).
 //  * moe_down_simple: out[t] += sum over the slots, in order, of Wdown_e y[t][s].
 //  Both take a shared expert along when one is given: its gate/up products as one more pair per
-//  token with weight 1, its down product added to the token's sum times the token's gate.
+//  token with weight 1, its down product added to the token's sum times the token's gate (or, without
+//  gates, times one factor).
 //  * scale_rows: y[t] *= f[t].
 //
 // These are the true 32-bit kernels and the general path of the bfloat16 engine; float32
@@ -144,30 +146,37 @@ constexpr int MAX_GROUPS = 64;
 
 __global__ void __launch_bounds__(WARPS * 32)
 router_choose_kernel(const float* logits, int stride, int num_tokens, int total, int top,
-                     const float* __restrict__ correction, int groups, int keep,
-                     int* __restrict__ ids, float* __restrict__ weights) {
+                     const float* __restrict__ correction, int groups, int keep, int sigmoid, int best_of,
+                     int normalize, float factor, int* __restrict__ ids, float* __restrict__ weights) {
     __shared__ float choice[WARPS][MAX_ROUTED];
     __shared__ float group_best[WARPS][MAX_GROUPS];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x * WARPS + warp;
     if (t >= num_tokens) return;
     const float* z = logits + (size_t)t * stride;
-    float m = -INFINITY;
-    for (int e = lane; e < total; e += 32) m = fmaxf(m, z[e]);
-    const float z_max = warp_max(m);
-    float acc = 0.0f;
-    for (int e = lane; e < total; e += 32) acc += expf(z[e] - z_max);
-    const float z_sum = warp_sum(acc);
+    float z_max = 0.0f, z_sum = 1.0f;
+    if (!sigmoid) {
+        float m = -INFINITY;
+        for (int e = lane; e < total; e += 32) m = fmaxf(m, z[e]);
+        z_max = warp_max(m);
+        float acc = 0.0f;
+        for (int e = lane; e < total; e += 32) acc += expf(z[e] - z_max);
+        z_sum = warp_sum(acc);
+    }
+    auto score = [&](int e) { return sigmoid ? sigmoidf_(z[e]) : expf(z[e] - z_max) / z_sum; };
     float* c = choice[warp];
-    for (int e = lane; e < total; e += 32) c[e] = expf(z[e] - z_max) / z_sum + (correction ? correction[e] : 0.0f);
+    for (int e = lane; e < total; e += 32) c[e] = score(e) + (correction ? correction[e] : 0.0f);
     __syncwarp();
     if (groups > 1 && keep < groups) {
         const int per = total / groups;
         float* gb = group_best[warp];
         for (int g = lane; g < groups; g += 32) {
-            float b = -INFINITY;
-            for (int e = g * per; e < (g + 1) * per; ++e) b = fmaxf(b, c[e]);
-            gb[g] = b;
+            float b = -INFINITY, b2 = -INFINITY;       // the largest and the one behind it
+            for (int e = g * per; e < (g + 1) * per; ++e) {
+                b2 = fmaxf(b2, fminf(b, c[e]));
+                b = fmaxf(b, c[e]);
+            }
+            gb[g] = best_of > 1 && per > 1 ? b + b2 : b;
         }
         __syncwarp();
         // a group stays if fewer than `keep` groups come before it (a larger value, or the same and a lower index)
@@ -179,6 +188,7 @@ router_choose_kernel(const float* logits, int stride, int num_tokens, int total,
         }
         __syncwarp();
     }
+    int mine = -1;                                     // the output of the slot that belongs to this lane (top <= 32)
     for (int s = 0; s < top; ++s) {
         float best = -INFINITY;
         int best_e = total;                           // larger than every index: loses every tie
@@ -193,13 +203,20 @@ router_choose_kernel(const float* logits, int stride, int num_tokens, int total,
             if (oe < total && (best_e == total || ov > best || (ov == best && oe < best_e))) { best = ov; best_e = oe; }
         }
         best_e = __shfl_sync(0xffffffffu, best_e, 0);
-        if (lane == 0) {
-            // fewer outputs left than slots (a configuration the caller refuses): the slot gets weight 0
-            ids[(size_t)t * top + s] = best_e < total ? best_e : 0;
-            weights[(size_t)t * top + s] = best_e < total ? expf(z[best_e] - z_max) / z_sum : 0.0f;
-            if (best_e < total) c[best_e] = -INFINITY;
-        }
+        if (lane == s && best_e < total) mine = best_e;
+        if (lane == 0 && best_e < total) c[best_e] = -INFINITY;
         __syncwarp();
+    }
+    // fewer outputs left than slots (a configuration the caller refuses): the slot gets weight 0
+    float w = mine >= 0 ? score(mine) : 0.0f;
+    if (normalize) {
+        float sum = 0.0f;                             // in the order of the slots
+        for (int s = 0; s < top; ++s) sum += __shfl_sync(0xffffffffu, w, s);
+        w /= sum + 1e-20f;
+    }
+    if (lane < top) {
+        ids[(size_t)t * top + lane] = mine >= 0 ? mine : 0;
+        weights[(size_t)t * top + lane] = w * factor;
     }
 }
 
@@ -228,6 +245,13 @@ moe_gate_up_simple_kernel(const TA* __restrict__ h, int h_stride, const TW* __re
     if (e >= experts) return;                         // an identity expert: nothing to multiply
     const float w = shared ? 1.0f : weights[ts];
     const TA* x = h + (size_t)(shared ? ts : ts / top) * h_stride;
+    if (!act_is_gated(act)) {                         // an expert is its ff up rows
+        float u, unused;
+        lane_dots(x, w_gate_up + ((size_t)e * ff + f) * width, (const TW*)nullptr, width, lane, u, unused);
+        u = warp_sum(u);
+        if (lane == 0) y[(size_t)ts * ff + f] = from_f32<TA>(w * unary_activation(act, u));
+        return;
+    }
     // an expert's 2 ff rows: strips of 8 gate rows and their 8 up rows, or all gate rows and then all up rows
     const size_t gate_row = interleaved ? (size_t)(f >> 3) * 16 + (f & 7) : (size_t)f;
     const size_t up_row = interleaved ? gate_row + 8 : (size_t)ff + f;
@@ -252,7 +276,7 @@ moe_down_simple_kernel(const TA* __restrict__ y, const TW* __restrict__ w_down,
                        float* __restrict__ out, int out_stride, const TA* __restrict__ y_shared,
                        const TW* __restrict__ w_shared_down, const float* __restrict__ shared_gate,
                        int shared_ff, int experts, const TA* __restrict__ h, int h_stride,
-                       const float* __restrict__ weights) {
+                       const float* __restrict__ weights, float shared_factor) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x;
     const int n = blockIdx.y * WARPS + warp;
@@ -275,7 +299,7 @@ moe_down_simple_kernel(const TA* __restrict__ y, const TW* __restrict__ w_down,
         const TW* wd = w_shared_down + (size_t)n * shared_ff;
         float acc, unused;
         lane_dots(ys, wd, (const TW*)nullptr, shared_ff, lane, acc, unused);
-        total += warp_sum(acc) * shared_gate[t];
+        total += warp_sum(acc) * (shared_gate ? shared_gate[t] : shared_factor);
     }
     if (lane == 0) out[(size_t)t * out_stride + n] += total;
 }
@@ -311,18 +335,21 @@ extern "C" int ti_router_topk(const float* logits, int stride, int num_tokens, i
 }
 
 // `total` router outputs in `groups` equal groups of which `keep` may be chosen from (groups = 1: no groups);
-// `correction` (may be null) is added to the scores for the choice alone.
+// `correction` (may be null) is added to the scores for the choice alone.  `sigmoid`: scores are sigmoids, else a
+// softmax; a group counts the sum of its `best_of` (1 or 2) largest values; `normalize`: weights are divided by
+// their sum (+ 1e-20); `factor` multiplies them.
 extern "C" int ti_router_choose(const float* logits, int stride, int num_tokens, int total, int top,
-                                const float* correction, int groups, int keep, int* ids, float* weights,
-                                void* stream) {
+                                const float* correction, int groups, int keep, int sigmoid, int best_of,
+                                int normalize, float factor, int* ids, float* weights, void* stream) {
     if (num_tokens == 0) return 0;
     TI_REQUIRE(total >= 1 && total <= MAX_ROUTED, "router_choose: %d router outputs (at most %d)", total, MAX_ROUTED);
     TI_REQUIRE(groups >= 1 && groups <= MAX_GROUPS && total % groups == 0 && keep >= 1 && keep <= groups,
                "router_choose: %d outputs in %d groups of which %d are kept", total, groups, keep);
+    TI_REQUIRE(best_of == 1 || best_of == 2, "router_choose: a group's value is its largest or the sum of its two largest");
     TI_REQUIRE(top >= 1 && top <= MAX_TOP && top <= total / groups * keep,
                "router_choose: %d of %d outputs cannot be chosen", top, total / groups * keep);
     router_choose_kernel<<<(num_tokens + WARPS - 1) / WARPS, WARPS * 32, 0, (cudaStream_t)stream>>>(
-        logits, stride, num_tokens, total, top, correction, groups, keep, ids, weights);
+        logits, stride, num_tokens, total, top, correction, groups, keep, sigmoid, best_of, normalize, factor, ids, weights);
     return ti_check_launch("router_choose");
 }
 
@@ -353,14 +380,14 @@ extern "C" int ti_moe_down_simple(const void* y, int act_dtype, const void* w_do
                                   float* out, int out_stride, const void* y_shared,
                                   const void* w_shared_down, const float* shared_gate, int shared_ff,
                                   int experts, const void* h, int h_stride, const float* weights,
-                                  void* stream) {
+                                  float shared_factor, void* stream) {
     if (num_tokens == 0) return 0;
     dim3 grid(num_tokens, (width + WARPS - 1) / WARPS);
     cudaStream_t s = (cudaStream_t)stream;
 #define CALL(TA, TW)                                                                         \
     moe_down_simple_kernel<TA, TW><<<grid, WARPS * 32, 0, s>>>(                               \
         (const TA*)y, (const TW*)w_down, ids, top, width, ff, out, out_stride, (const TA*)y_shared, \
-        (const TW*)w_shared_down, shared_gate, shared_ff, experts, (const TA*)h, h_stride, weights)
+        (const TW*)w_shared_down, shared_gate, shared_ff, experts, (const TA*)h, h_stride, weights, shared_factor)
     TI_DISPATCH_AW(act_dtype, w_dtype, CALL)
 #undef CALL
     return ti_check_launch("moe_down_simple");

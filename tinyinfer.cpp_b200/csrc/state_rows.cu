@@ -19,6 +19,7 @@
 //    tanh_norm_pair: such a norm's rows are added to the residual and the sum passes a second such norm in the
 //    same launch (the norm behind one sublayer and the norm in front of the next).
 //  * cap_rows: x = cap tanh(x / cap), in place.
+//  * unary_rows: y = act(x) with an activation of one value (glu.cuh).
 //  * add_row: x[t] += row for every row of x.
 //  * embed_bigram: the embedding row of a token plus a row of a second table that a hash of the token and
 //    the one before it chooses; the request keeps its last token.
@@ -359,6 +360,12 @@ __global__ void cap_rows_kernel(float* __restrict__ x, size_t total, float cap) 
     if (i < total) x[i] = cap * tanhf(x[i] / cap);
 }
 
+template <typename TO>
+__global__ void unary_rows_kernel(const float* x, size_t total, int kind, TO* __restrict__ out) {
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i < total) out[i] = from_f32<TO>(unary_activation(kind, x[i]));
+}
+
 __global__ void add_row_kernel(float* __restrict__ x, int stride, const float* __restrict__ row, int cols, size_t total) {
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= total) return;
@@ -536,6 +543,17 @@ extern "C" int ti_cap_rows(float* x, long long total, float cap, void* stream) {
     TI_REQUIRE(cap > 0.0f, "cap_rows: the cap must be positive");
     cap_rows_kernel<<<(unsigned)((total + 255) / 256), 256, 0, (cudaStream_t)stream>>>(x, (size_t)total, cap);
     return ti_check_launch("cap_rows");
+}
+
+extern "C" int ti_unary_rows(const float* x, long long total, int kind, void* out, int out_dtype, void* stream) {
+    if (total == 0) return 0;
+    TI_REQUIRE(kind == ACT_RELU2, "unary_rows: activation kind %d", kind);
+    const unsigned blocks = (unsigned)((total + 255) / 256);
+    cudaStream_t s = (cudaStream_t)stream;
+    if (out_dtype == TI_BF16) unary_rows_kernel<bf16><<<blocks, 256, 0, s>>>(x, (size_t)total, kind, (bf16*)out);
+    else if (out_dtype == TI_F32) unary_rows_kernel<float><<<blocks, 256, 0, s>>>(x, (size_t)total, kind, (float*)out);
+    else return ti_fail("unary_rows: output dtype code %d", out_dtype);
+    return ti_check_launch("unary_rows");
 }
 
 extern "C" int ti_add_row(float* x, int stride, const float* row, int rows, int cols, void* stream) {

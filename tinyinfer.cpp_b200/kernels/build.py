@@ -30,14 +30,14 @@ LIBRARIES = {
     # tensor-core kernels of the attention with a distance bias and of the routed feed-forward
     "bf16_gated": ["common.cu", "attn_gated_bias_tc.cu", "attn_bias_prefill_tc.cu", "moe_grouped.cu"],
     # attention with optional parts (chunks, caps, sinks, gates, shared rows) and the recurrent mixer
-    "mixers": ["common.cu", "attn_options.cu", "wkv.cu"],
+    "mixers": ["common.cu", "attn_options.cu", "head_rows.cu", "wkv.cu"],
     "bf16_mixers": ["common.cu", "attn_options_tc.cu"],
     # recurrent mixers with a matrix state
     "state": ["common.cu", "matrix_state.cu", "matrix_state_decayed.cu"],
     # recurrences per channel and the gates and decays in front of them
     "channels": ["common.cu", "channel_recurrence.cu"],
     # short convolutions over time, norms in groups and without statistics, depth sums, gated activations
-    "rows": ["common.cu", "state_rows.cu"],
+    "rows": ["common.cu", "state_rows.cu", "layer_norm.cu"],
 }
 
 # libraries that parts bring themselves: name -> (absolute source paths, include folders)

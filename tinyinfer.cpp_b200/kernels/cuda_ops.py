@@ -12,6 +12,8 @@ pack_gate_up(gate, up) -> w'                 the stacked gate/up weight
 embed(table, token_ids, out)                 out[t] = float32(table[token_ids[t]])
 rmsnorm(x, weight, eps, out, rows=None)      out[r] = norm(x[rows[r]] or x[r]), rounded to out.dtype
 linear(a, w, out, accumulate=False)          out (+)= a @ w.T in float32 (or through a gate into a residual)
+linear_unary(h, w, kind, out)                out = act(h @ w.T) with an activation of one value
+unary_ffn(h, w_up, w_down, residual, kind)   residual += act(h @ w_up.T) @ w_down.T
 linear_xielu(h, w, ap, aq, out)              out = xielu(h @ w.T), one launch for few rows
 glu_ffn(h, w_gate_up, w_down, residual, ...) residual += act(gate, up) @ w_down.T with a gated activation
 gate_up_swiglu(h, w, out)                    out = silu(h @ gate.T) * (h @ up.T)
@@ -218,11 +220,11 @@ class CudaOps(MixerOps, StateOps):
         c.ti_attention_bias_simple.argtypes = [_vp, _i, _vp, _vp, _vp, _vp, _i, _vp, _i, _i, _i, _i, _i, _i,
                                                _i, _i, _i, _i, _f, _vp, _i, _vp, _i, _vp, _vp, _vp]
         c.ti_router_topk.argtypes = [_vp, _i, _i, _i, _i, _i, _vp, _vp, _vp, _i, _vp]
-        c.ti_router_choose.argtypes = [_vp, _i, _i, _i, _i, _vp, _i, _i, _vp, _vp, _vp]
+        c.ti_router_choose.argtypes = [_vp, _i, _i, _i, _i, _vp, _i, _i, _i, _i, _i, _f, _vp, _vp, _vp]
         c.ti_moe_gate_up_simple.argtypes = [_vp, _i, _i, _vp, _i, _i, _vp, _vp, _i, _i, _i, _i, _vp, _vp, _i, _i,
                                             _vp, _i, _f, _f, _i, _vp]
         c.ti_moe_down_simple.argtypes = [_vp, _i, _vp, _i, _vp, _i, _i, _i, _i, _vp, _i, _vp, _vp, _vp, _i, _i, _vp,
-                                         _i, _vp, _vp]
+                                         _i, _vp, _f, _vp]
         c.ti_scale_rows.argtypes = [_vp, _i, _i, _vp, _i, _i, _vp]
 
     @property
@@ -234,8 +236,9 @@ class CudaOps(MixerOps, StateOps):
             b.ti_gemm_skinny.argtypes = [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp]
             b.ti_gemm_skinny_supported.argtypes = [_i, _i, _i, _i, _i]
             b.ti_gemm_skinny_xielu.argtypes = [_vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _f, _vp]
+            b.ti_gemm_skinny_unary.argtypes = [_vp, _vp, _vp] + [_i] * 7 + [_vp]
             b.ti_gemm_skinny_gated.argtypes = [_vp, _vp, _vp] + [_i] * 6 + [_vp, _i, _vp, _f, _vp]
-            b.ti_gemm_skinny_pair.argtypes = [_vp, _vp, _vp, _vp] + [_i] * 8 + [_f, _f, _vp, _vp, _vp] + [_i] * 4 + [_vp]
+            b.ti_gemm_skinny_pair.argtypes = [_vp, _vp, _vp, _vp] + [_i] * 8 + [_f, _f, _vp, _vp, _vp] + [_i] * 5 + [_vp]
             b.ti_gemm_tcgen05_few_gated.argtypes = [_vp, _vp, _vp] + [_i] * 6 + [_vp, _vp, _vp, _i, _vp, _f, _vp, _vp]
             b.ti_gemm_tcgen05_gated.argtypes = [_vp, _vp, _vp] + [_i] * 6 + [_vp, _vp, _i, _vp, _f, _vp, _vp]
             b.ti_gemm_tcgen05_2sm_gated.argtypes = [_vp, _vp, _vp] + [_i] * 6 + [_vp, _i, _vp, _f, _vp, _vp]
@@ -520,14 +523,14 @@ class CudaOps(MixerOps, StateOps):
             return False
         a2, w2, out2 = held
         m, k = a.shape
-        if a2.shape != a.shape or not (glu is not None or self._pairable(a, w)):
+        if a2.shape[0] != a.shape[0] or not (glu is not None or self._pairable(a, w)):
             return False
         self._pending_pair = None
         kind, limit, alpha = glu if glu is not None else (-1, 0.0, 0.0)
         self._ok(self.bf16.ti_gemm_skinny_pair(
             a.data_ptr(), w.data_ptr(), _ptr(out), _ptr(out_act), m, w.shape[0], k, a.stride(0), w.stride(0),
             out.stride(0) if out is not None else 0, out_act.stride(0) if out_act is not None else 0, kind, float(limit),
-            float(alpha), a2.data_ptr(), w2.data_ptr(), out2.data_ptr(), w2.shape[0], a2.stride(0), w2.stride(0),
+            float(alpha), a2.data_ptr(), w2.data_ptr(), out2.data_ptr(), w2.shape[0], w2.shape[1], a2.stride(0), w2.stride(0),
             out2.stride(0), self._stream()), self.bf16)
         return True
 
@@ -586,17 +589,20 @@ class CudaOps(MixerOps, StateOps):
             self._stream()))
 
     def _linear_gated_sum(self, a, w, target):
-        """``x += scale * sigmoid(gate + bias) * (a @ w.T)`` for a ``parts.base.GatedSum``: in the product's
-        epilogue where a tensor-core product takes the operands, else behind it."""
+        """``x += scale * sigmoid(gate + bias) * (a @ w.T)`` for a ``parts.base.GatedSum`` (without a gate ``x +=
+        scale * (a @ w.T)``): in the product's epilogue where a tensor-core product takes the operands, else
+        behind it."""
         x, gate, bias = target.x, target.gate, target.bias
         m, k = a.shape
         n = w.shape[0]
-        _need(w.shape[1] == k and tuple(x.shape) == tuple(gate.shape) == (m, n) and bias.numel() == n
-              and x.dtype == gate.dtype == bias.dtype == torch.float32 and bias.is_contiguous()
-              and x.stride(1) == gate.stride(1) == 1, "linear: a gated sum of float32 rows of the product's shape")
+        _need(w.shape[1] == k and tuple(x.shape) == (m, n) and x.dtype == torch.float32 and x.stride(1) == 1,
+              "linear: a gated sum of float32 rows of the product's shape")
+        _need(gate is None or (tuple(gate.shape) == (m, n) and bias.numel() == n and gate.dtype == bias.dtype == torch.float32
+                               and bias.is_contiguous() and gate.stride(1) == 1),
+              "linear: a gated sum's gate and bias")
         if (self.fuse_gated_sums and a.dtype == w.dtype == torch.bfloat16 and a.stride(1) == w.stride(1) == 1
                 and a.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0):
-            args = (gate.data_ptr(), gate.stride(0), bias.data_ptr(), float(target.scale))
+            args = (_ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(bias), float(target.scale))
             sizes = (a.data_ptr(), w.data_ptr(), x.data_ptr(), m, n, k, a.stride(0), w.stride(0), x.stride(0))
             status, stream = self.status.data_ptr(), self._stream()
             few = self._few_tc_scratch(a, w, 1)
@@ -607,8 +613,8 @@ class CudaOps(MixerOps, StateOps):
             if self.bf16.ti_gemm_skinny_supported(m, n, k, a.stride(0), w.stride(0)):
                 self._ok(self.bf16.ti_gemm_skinny_gated(*sizes, *args, stream), self.bf16)
                 return
-            if (m > 64 and x.data_ptr() % 16 == 0 and gate.data_ptr() % 16 == 0 and gate.stride(0) % 4 == 0
-                    and bias.data_ptr() % 16 == 0
+            if (m > 64 and x.data_ptr() % 16 == 0
+                    and (gate is None or (gate.data_ptr() % 16 == 0 and gate.stride(0) % 4 == 0 and bias.data_ptr() % 16 == 0))
                     and self.bf16.ti_gemm_tcgen05_supported(m, n, k, a.stride(0), w.stride(0), x.stride(0), 1)):
                 if self._tc_gemm(m, n) is self.bf16.ti_gemm_tcgen05_2sm:
                     self._ok(self.bf16.ti_gemm_tcgen05_2sm_gated(*sizes, *args, status, stream), self.bf16)
@@ -647,6 +653,41 @@ class CudaOps(MixerOps, StateOps):
         self.linear(h, w_gate_up, gu)
         self._ok(self.core.ti_swiglu(gu.data_ptr(), m, inter, int(interleaved), out.data_ptr(),
                                      _code(out, "swiglu"), self._stream()))
+
+    def linear_unary(self, h, w, kind, out):
+        """out = act(h @ w.T) in the activation dtype with an activation of one value (``state_ops.UNARY_KINDS``), in
+        the product's epilogue where a tensor-core product takes the operands, else behind it."""
+        from .state_ops import UNARY_KINDS
+        m, k = h.shape
+        n = w.shape[0]
+        _need(w.shape[1] == k and tuple(out.shape) == (m, n) and out.dtype == h.dtype
+              and h.stride(1) == w.stride(1) == out.stride(1) == 1, "linear_unary: shapes do not agree")
+        if h.dtype == w.dtype == torch.bfloat16 and h.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0:
+            if self.bf16.ti_gemm_skinny_supported(m, n, k, h.stride(0), w.stride(0)):
+                self._ok(self.bf16.ti_gemm_skinny_unary(h.data_ptr(), w.data_ptr(), out.data_ptr(), m, n, k, h.stride(0),
+                                                        w.stride(0), out.stride(0), UNARY_KINDS[kind], self._stream()),
+                         self.bf16)
+                return
+            if (m > 64 and n % 8 == 0 and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0
+                    and self.bf16.ti_gemm_tcgen05_supported(m, n, k, h.stride(0), w.stride(0), 0, 0)):
+                self._ok(self.bf16.ti_gemm_tcgen05_glu(
+                    h.data_ptr(), w.data_ptr(), out.data_ptr(), m, n, k, h.stride(0), w.stride(0), out.stride(0),
+                    UNARY_KINDS[kind], 0.0, 0.0, self.status.data_ptr(), self._stream()), self.bf16)
+                return
+        z = torch.empty((m, n), dtype=torch.float32, device=h.device)
+        self.linear(h, w, z)
+        if out.is_contiguous():
+            self.unary_rows(z, kind, out)
+        else:
+            y = torch.empty((m, n), dtype=out.dtype, device=h.device)
+            self.unary_rows(z, kind, y)
+            out.copy_(y)
+
+    def unary_ffn(self, h, w_up, w_down, residual, kind):
+        """residual += act(h Wup^T) Wdown^T with an activation of one value; ``residual`` may be a ``GatedSum``."""
+        y = torch.empty((h.shape[0], w_up.shape[0]), dtype=h.dtype, device=h.device)
+        self.linear_unary(h, w_up, kind, y)
+        self.linear(y, w_down, residual, accumulate=True)
 
     def linear_xielu(self, h, w, ap, aq, out):
         """out = xielu(h @ w.T) in the activation dtype: ``ap z^2 + z/2`` where ``z > 0``, ``aq (exp(z) -
@@ -1158,7 +1199,12 @@ class CudaOps(MixerOps, StateOps):
     def pack_experts(self, gate, up, down):
         """The stacked weights of a routed feed-forward (``[experts, ff, width]`` twice and
         ``[experts, width, ff]``) in the layout the kernels want: an expert's gate and up rows as
-        one matrix (strips of 8 and 8 where the sizes allow, for the SwiGLU epilogues)."""
+        one matrix (strips of 8 and 8 where the sizes allow, for the SwiGLU epilogues).  ``gate`` None: experts
+        without a gate, whose first matrix is the up rows."""
+        if gate is None:
+            _need(up.dtype == down.dtype, "pack_experts: one dtype for all experts")
+            _code(up, "pack_experts")
+            return {"gate_up": up.contiguous(), "down": down.contiguous(), "interleaved": False, "gated": False}
         _need(gate.dtype == up.dtype == down.dtype, "pack_experts: one dtype for all experts")
         _code(gate, "pack_experts")
         experts, ff, width = gate.shape
@@ -1168,7 +1214,7 @@ class CudaOps(MixerOps, StateOps):
             gate_up = gate_up.reshape(experts, 2 * ff, width).contiguous()
         else:
             gate_up = torch.cat([gate, up], dim=1).contiguous()
-        return {"gate_up": gate_up, "down": down.contiguous(), "interleaved": interleaved}
+        return {"gate_up": gate_up, "down": down.contiguous(), "interleaved": interleaved, "gated": True}
 
     def router_topk(self, logits, experts, top, ids, weights, shared_gate=None, softmax=False):
         """Per row the ``top`` largest of the first ``experts`` logits (ties: the lower index):
@@ -1186,12 +1232,15 @@ class CudaOps(MixerOps, StateOps):
                                           weights.data_ptr(), _ptr(shared_gate), int(bool(softmax)),
                                           self._stream()))
 
-    def router_choose(self, logits, total, top, ids, weights, correction=None, groups=1, keep=1):
-        """Per row, from the first ``total`` float32 logits: scores ``s = softmax(logits)``; the
-        choice looks at ``s + correction`` (float32 ``[total]`` or None), only inside the ``keep`` of
-        ``groups`` equal groups of neighbouring outputs whose largest such value is largest, and
+    def router_choose(self, logits, total, top, ids, weights, correction=None, groups=1, keep=1, sigmoid=False,
+                      best_of=1, normalize=False, factor=1.0):
+        """Per row, from the first ``total`` float32 logits: scores ``s = softmax(logits)``, or with
+        ``sigmoid`` each logit's sigmoid; the choice looks at ``s + correction`` (float32 ``[total]`` or
+        None), only inside the ``keep`` of ``groups`` equal groups of neighbouring outputs with the largest
+        value, a group's value being its largest such sum or, ``best_of`` 2, its two largest added, and
         takes the ``top`` largest there (ties: the lower index).  ``ids`` int32 and ``weights``
-        float32 ``[rows, top]``: the chosen outputs and their ``s``, not renormalised."""
+        float32 ``[rows, top]``: the chosen outputs and their ``s``, with ``normalize`` divided by their sum
+        (+ 1e-20), times ``factor``."""
         t = logits.shape[0]
         _need(logits.dtype == torch.float32 and logits.stride(1) == 1 and logits.shape[1] >= total,
               "router_choose: float32 logits")
@@ -1201,7 +1250,8 @@ class CudaOps(MixerOps, StateOps):
               and weights.is_contiguous() and tuple(ids.shape) == tuple(weights.shape) == (t, top),
               "router_choose: ids int32 and weights float32, [rows, top]")
         self._ok(self.core.ti_router_choose(logits.data_ptr(), logits.stride(0), t, int(total), int(top),
-                                            _ptr(correction), int(groups), int(keep), ids.data_ptr(),
+                                            _ptr(correction), int(groups), int(keep), int(bool(sigmoid)), int(best_of),
+                                            int(bool(normalize)), float(factor), ids.data_ptr(),
                                             weights.data_ptr(), self._stream()))
 
     def routed_experts(self, h, w, ids, weights, residual, shared=None, act=None, identity=False):
@@ -1212,26 +1262,37 @@ class CudaOps(MixerOps, StateOps):
         it inside the experts' two launches.  ``act`` (may be None: silu) names another gated
         activation, ``(kind, limit, alpha)`` as ``glu_rows`` takes them; the pair's weight then
         scales the expert's output, residual[t] += w Wdown_e act(g, u), and there is no ``shared``.
+        Experts without a gate (``pack_experts(None, ...)``) take an activation of one value, residual[t] += w
+        Wdown_e act(u); their ``shared`` is ``(w_up, w_down, factor)``, residual[t] += factor Wdown act(Wup h[t]).
         ``identity``: an index at or behind the number of stacked experts names an identity expert,
         whose output is the token's input, residual[t] += w h[t]."""
         self._routed(h, w, ids, weights, residual, shared, act, identity)
 
-    def _shared_expert(self, h, shared, residual):
+    def _shared_expert(self, h, shared, residual, act=None):
         w_gate_up, w_down, gate = shared
+        if not isinstance(gate, torch.Tensor):       # no gate of either sort: one factor for all tokens
+            from ..parts.base import GatedSum
+            self.unary_ffn(h, w_gate_up, w_down, residual if gate == 1.0 else GatedSum(residual, None, None, gate), act[0])
+            return
         y = torch.empty((h.shape[0], w_down.shape[1]), dtype=h.dtype, device=h.device)
         self.gate_up_swiglu(h, w_gate_up, y)
         self.scale_rows(y, gate)
         self.linear(y, w_down, residual, accumulate=True)
 
     def _routed(self, h, w, ids, weights, residual, shared, act=None, identity=False):
-        from .state_ops import GLU_KINDS
-        act_kind, act_limit, act_alpha = (0, 0.0, 0.0) if act is None else (GLU_KINDS[act[0]], float(act[1]), float(act[2]))
-        _need(act_kind == 0 or shared is None, "routed_experts: a shared expert rides only with the silu activation")
+        from .state_ops import GLU_KINDS, UNARY_KINDS
+        gated = bool(w.get("gated", True))
+        kinds = GLU_KINDS if gated else UNARY_KINDS
+        act_kind, act_limit, act_alpha = (0, 0.0, 0.0) if act is None else (kinds[act[0]], float(act[1]), float(act[2]))
+        _need(gated or act is not None, "routed_experts: experts without a gate need an activation of one value")
+        _need(act_kind == 0 or not gated or shared is None, "routed_experts: a shared expert rides only with the silu activation")
+        _need(gated or shared is None or not isinstance(shared[2], torch.Tensor), "routed_experts: one factor for the shared expert")
         t, width = h.shape
         top = ids.shape[1]
         experts, ff = w["down"].shape[0], w["down"].shape[2]
         gate_up, interleaved = w["gate_up"], int(w["interleaved"])
-        _need(gate_up.shape == (experts, 2 * ff, width) and w["down"].shape == (experts, width, ff),
+        first = 2 * ff if gated else ff              # rows of an expert's first matrix
+        _need(gate_up.shape == (experts, first, width) and w["down"].shape == (experts, width, ff),
               "routed_experts: expert shapes do not agree")
         _need(residual.dtype == torch.float32 and residual.stride(1) == 1 and tuple(residual.shape) == (t, width),
               "routed_experts: float32 residual")
@@ -1241,8 +1302,8 @@ class CudaOps(MixerOps, StateOps):
                 and h.stride(0) % 8 == 0 and h.data_ptr() % 16 == 0
                 and self.gated.ti_moe_grouped_supported(width, ff, experts)):
             pairs = t * top
-            if (self.tcgen05_experts_from is not None and pairs >= self.tcgen05_experts_from and interleaved
-                    and ff % 16 == 0 and width % 8 == 0):
+            if (self.tcgen05_experts_from is not None and pairs >= self.tcgen05_experts_from
+                    and (interleaved or not gated) and ff % 16 == 0 and width % 8 == 0):
                 # every expert's pairs in whole tiles of 128 rows, the rows of h times their weights
                 # gathered in that order, two grouped tcgen05 products (the first with SwiGLU in its
                 # epilogue), and the pairs' rows added per token; with another activation the rows of h
@@ -1261,7 +1322,7 @@ class CudaOps(MixerOps, StateOps):
                                                 a.data_ptr(), self._stream()), g)
                 y = torch.empty((max_rows, ff), dtype=torch.bfloat16, device=h.device)
                 self._ok(self.bf16.ti_gemm_tcgen05_grouped_glu(
-                    a.data_ptr(), gate_up.data_ptr(), y.data_ptr(), max_rows, 2 * ff, width, width, width, ff,
+                    a.data_ptr(), gate_up.data_ptr(), y.data_ptr(), max_rows, first, width, width, width, ff,
                     experts, group_of_tile.data_ptr(), tiles_m.data_ptr(), act_kind, act_limit, act_alpha,
                     self.status.data_ptr(), self._stream()), self.bf16)
                 out_rows = torch.empty((max_rows, width), dtype=torch.float32, device=h.device)
@@ -1275,7 +1336,7 @@ class CudaOps(MixerOps, StateOps):
                                                ids.data_ptr() if identity else None, experts, weights.data_ptr(),
                                                h.data_ptr(), h.stride(0), self._stream()), g)
                 if shared is not None:
-                    self._shared_expert(h, shared, residual)
+                    self._shared_expert(h, shared, residual, act)
                 return
             ints = torch.empty(pairs + 3 * (pairs // 64 + experts) + 1, dtype=torch.int32, device=h.device)
             y_sorted = torch.empty((pairs, ff), dtype=torch.bfloat16, device=h.device)
@@ -1288,22 +1349,26 @@ class CudaOps(MixerOps, StateOps):
                 int(bool(identity)), self._stream()), self.gated)
             self.launches += 3
             if shared is not None:
-                self._shared_expert(h, shared, residual)
+                self._shared_expert(h, shared, residual, act)
             return
         # the CUDA-core kernels; a small shared expert of the experts' weight dtype rides along (two
         # launches instead of five).  A large one does not: these kernels fetch an expert's rows once
         # per pair, which for an expert that every token uses means once per token (measured at
         # batch 8: 5,784 -> 5,277 tok/s with a shared expert of 2,048 x 4,096 riding along)
         ride = (shared is not None and shared[0].dtype == gate_up.dtype and shared[1].dtype == gate_up.dtype
-                and shared[0].is_contiguous() and shared[1].is_contiguous() and shared[2].dtype == torch.float32
+                and shared[0].is_contiguous() and shared[1].is_contiguous()
+                and (not gated or shared[2].dtype == torch.float32)
                 and shared[1].shape[1] * width <= self.shared_rides_to)
         y_sh = sgu = sdown = sgate = None
         s_ff = s_inter = 0
+        s_factor = 1.0
         if ride:
             sgu, sdown, sgate = shared
+            if not gated:
+                s_factor, sgate = float(sgate), None
             s_ff, s_inter = sdown.shape[1], int(bool(getattr(sgu, "_ti_interleaved", False)))
-            _need(tuple(sgu.shape) == (2 * s_ff, width) and tuple(sdown.shape) == (width, s_ff)
-                  and sgate.shape[0] == t and sgate.is_contiguous(), "routed_experts: the shared expert's shapes")
+            _need(tuple(sgu.shape) == ((2 if gated else 1) * s_ff, width) and tuple(sdown.shape) == (width, s_ff)
+                  and (sgate is None or (sgate.shape[0] == t and sgate.is_contiguous())), "routed_experts: the shared expert's shapes")
             y_sh = torch.empty((t, s_ff), dtype=h.dtype, device=h.device)
         y = torch.empty((t, top, ff), dtype=h.dtype, device=h.device)
         self._ok(self.core.ti_moe_gate_up_simple(
@@ -1315,9 +1380,9 @@ class CudaOps(MixerOps, StateOps):
             y.data_ptr(), _code(y, "routed_experts"), w["down"].data_ptr(), _code(w["down"], "routed_experts"),
             ids.data_ptr(), t, top, width, ff, residual.data_ptr(), residual.stride(0), _ptr(y_sh), _ptr(sdown),
             _ptr(sgate), s_ff, experts if identity else 1 << 30, h.data_ptr(), h.stride(0), weights.data_ptr(),
-            self._stream()))
+            s_factor, self._stream()))
         if shared is not None and not ride:
-            self._shared_expert(h, shared, residual)
+            self._shared_expert(h, shared, residual, act)
 
     def scale_rows(self, y, factors):
         """y[r] *= factors[r] (float32 factors), in place."""

@@ -1,4 +1,4 @@
-"""Bindings of the kernels in ``csrc/attn_options.cu`` and ``csrc/wkv.cu`` (library ``mixers``):
+"""Bindings of the kernels in ``csrc/attn_options.cu``, ``csrc/head_rows.cu`` and ``csrc/wkv.cu`` (library ``mixers``):
 attention with optional parts (chunk or window mask, a score factor per head, a cap on the score,
 a sink in the softmax, an output gate per head or per element, keys and values read from one
 shared row), the kernels that prepare its heads, and a recurrent mixer with a matrix state.
@@ -12,6 +12,8 @@ latent_prepare(proj, ...)            normed latent + turned key part as one cach
                                      and turned query parts out
 qkv_turn_store(proj, ...)            norms of whole rows or none, queries and keys turned, values mixed with another layer's, values turned by frequencies of
                                      their own, keys/values into pages, queries out
+heads_prepare_store(proj, ...)       heads by themselves: bias, norm in front of the turn, turn, norm behind it, a
+                                     factor of the position on queries, keys/values into pages, queries out
 slice_rmsnorm(x, weight, eps, out)   RMS norm of a column slice of a product
 turn_rows(x, step, rotation, ...)    finished rows' heads turned by plus or minus their position, times
                                      sigmoid(gate)
@@ -87,6 +89,8 @@ class MixerOps:
                                             _i, _i, _i, _vp, _vp, _i, _vp, _vp]
             b.ti_qkv_turn_store.argtypes = [_vp, _i, _i, _f, _vp, _vp, _vp, _i, _f, _vp, _i, _i, _f, _vp, _i, _i, _vp, _vp, _vp, _i, _vp, _i, _i, _i,
                                             _i, _i, _i, _i, _i, _i, _vp, _i, _vp, _vp]
+            b.ti_heads_prepare_store.argtypes = [_vp, _i, _vp, _vp, _vp, _i, _i, _f, _vp, _i, _i, _f, _f, _i, _i, _vp, _vp,
+                                                 _vp, _i, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _i, _vp, _vp]
             b.ti_slice_rmsnorm.argtypes = [_vp, _i, _i, _i, _vp, _f, _vp, _i, _vp]
             b.ti_turn_rows.argtypes = [_vp, _i, _vp, _vp, _i, _i, _f, _vp, _i, _i, _i, _i, _vp, _vp]
             b.ti_head_project.argtypes = [_vp, _i, _i, _i, _vp, _i, _i, _i, _vp, _i, _i, _i, _i, _i, _vp]
@@ -239,6 +243,50 @@ class MixerOps:
             pages.data_ptr(), _CODE[pages.dtype], pages.shape[0], cache.page_size, int(bool(cache.writes)), t,
             num_heads, num_kv_heads, dk, dv, q_out.data_ptr(), _CODE[q_out.dtype], self.status.data_ptr(),
             self._stream()))
+
+    def heads_prepare_store(self, proj, rotation, step, cache, q_out, num_heads, num_kv_heads, dk, dv, *, bias=None,
+                            pre_norm=None, post_norm_eps=None, query_factor=None, values_from_keys=False):
+        """From the float32 product ``proj`` (columns: queries, keys, values, then anything else), each query
+        and key head by itself: ``bias`` (float32 per column of the three, or None) is added; with ``pre_norm
+        = (q_weight, k_weight, eps)`` the head is RMS-normed with a weight of ``dk`` elements that all heads share
+        (or None); its first ``rotation.rotary_dim`` elements are turned by the token's position (kind
+        ``interleaved``, ``neox`` or ``none``; sine and cosine times ``rotation.scale``); with
+        ``post_norm_eps`` it is RMS-normed again, without a weight; a query is multiplied by ``1 + coef
+        ln(floor((position + 1) / every) + 1)`` for ``query_factor = (coef, every)``.  Keys and values go into
+        the token's page (if the cache slot is written), queries into ``q_out``.  ``values_from_keys``: there
+        are no value columns, the values are the key columns (with their bias) as they are."""
+        t = proj.shape[0]
+        pages, bt = cache.pages, cache.block_table
+        nq, nk = num_heads * dk, num_kv_heads * dk
+        nv = 0 if values_from_keys else num_kv_heads * dv
+        rot = 0 if rotation.kind == "none" else int(rotation.rotary_dim)
+        self._must(rot == 0 or (rotation.kind in self._LAYOUTS and rotation.inv_freq is not None
+                                and rotation.inv_freq.dtype == torch.float32 and rotation.inv_freq.shape[0] >= rot // 2),
+                   "heads_prepare_store: the rotation needs a known pairing and rotary_dim/2 float32 frequencies")
+        self._must(proj.dtype == torch.float32 and proj.stride(1) == 1
+                   and proj.shape[1] >= nq + (nk + nv if cache.writes else 0),
+                   "heads_prepare_store: the product must be float32 and hold all heads")
+        self._must(bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.shape[0] == nq + nk + nv),
+                   "heads_prepare_store: one float32 bias per column of queries, keys and values")
+        q_weight, k_weight, pre_eps = pre_norm if pre_norm is not None else (None, None, 0.0)
+        self._must(pre_norm is None or post_norm_eps is None or pre_eps == post_norm_eps,
+                   "heads_prepare_store: both norms have one eps")
+        for w in (q_weight, k_weight):
+            self._must(w is None or (w.dtype == torch.float32 and w.is_contiguous() and w.shape[0] == dk),
+                       "heads_prepare_store: a norm weight must be float32, one value per element of a head")
+        self._must(pages.is_contiguous() and pages[0].numel() == num_kv_heads * cache.page_size * (dk + dv),
+                   "heads_prepare_store: page layout")
+        self._must(bt.dtype == torch.int32 and bt.stride(1) == 1, "heads_prepare_store: block table int32")
+        self._must(q_out.is_contiguous() and tuple(q_out.shape) == (t, nq), "heads_prepare_store: q_out")
+        coef, every = query_factor if query_factor is not None else (0.0, 0)
+        self._mx(self.mixers.ti_heads_prepare_store(
+            proj.data_ptr(), proj.stride(0), _ptr(bias), _ptr(q_weight), _ptr(k_weight), int(pre_norm is not None),
+            int(post_norm_eps is not None), float(pre_eps if post_norm_eps is None else post_norm_eps),
+            _ptr(rotation.inv_freq) if rot else None, rot, self._LAYOUTS.get(rotation.kind, 0),
+            float(getattr(rotation, "scale", 1.0)), float(coef), int(every), int(bool(values_from_keys)),
+            step.positions.data_ptr(), step.req_of_tok.data_ptr(), bt.data_ptr(), bt.stride(0), pages.data_ptr(),
+            _CODE[pages.dtype], pages.shape[0], cache.page_size, int(bool(cache.writes)), t, num_heads, num_kv_heads, dk,
+            dv, q_out.data_ptr(), _CODE[q_out.dtype], self.status.data_ptr(), self._stream()))
 
     def turn_rows(self, x, step, rotation, num_heads, n, back=False, gate=None, out=None):
         """``out[t, h, :]`` is head ``h`` of row ``t`` of ``x`` (``[T, heads * n]``) with its first

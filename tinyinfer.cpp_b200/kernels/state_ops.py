@@ -1,5 +1,6 @@
 """Bindings of the kernels in ``csrc/matrix_state*.cu`` (library ``state``),
-``csrc/channel_recurrence.cu`` (library ``channels``) and ``csrc/state_rows.cu`` (library ``rows``): recurrent mixers with a float32 matrix state per head, short causal convolutions
+``csrc/channel_recurrence.cu`` (library ``channels``), ``csrc/state_rows.cu`` and ``csrc/layer_norm.cu`` (library
+``rows``): recurrent mixers with a float32 matrix state per head, short causal convolutions
 over time with their kept inputs, norms in groups, the depth-weighted mix of layer outputs, and
 gated activations with clamps.
 
@@ -16,6 +17,8 @@ low_rank_decay(low, a2, bias, tau, out)                        sigmoid(low a2^T 
 gated_recurrence(...)                                          a linear recurrence per channel with its gates
 tanh_norm(x, alpha, w, b, out | residual, rows)                tanh(alpha x) w + b, the norm without mean or variance
 tanh_norm_pair(y, ..., residual, ..., out)                     residual += norm1(y); out = norm2(residual)
+layer_norm(x, w, b, eps, out, rows)                            (x - mean) / sqrt(var + eps) w + b
+norm_sum(a, b, wa, wb, eps, target, then)                      x += scale (rms(a) wa + rms(b) wb), then a layer norm of x
 cap_rows(x, cap)                                               x = cap tanh(x / cap), in place
 add_row(x, row)                                                x[t] += row
 depth_mix(x, hist, index, weights)                             hist[index] = x; x = sum_j weights[j] hist[j]
@@ -35,6 +38,7 @@ _CODE = {torch.float32: 0, torch.bfloat16: 1}
 _vp, _i, _f, _ll = ctypes.c_void_p, ctypes.c_int, ctypes.c_float, ctypes.c_longlong
 
 GLU_KINDS = {"silu": 0, "clamped": 1, "gelu_tanh": 2}
+UNARY_KINDS = {"relu2": 16}              # activations of one value, of feed-forwards without a gate
 STATE_MODES = {"delta": 0, "gated_sum": 1, "decayed_sum": 2}
 GATE_ACTS = {"silu": 0, "sigmoid": 1}
 
@@ -123,6 +127,9 @@ class StateOps:
             b.ti_group_norm_rows.argtypes = [_vp, _vp, _vp, _i, _i, _i, _f, _vp, _i, _vp, _i, _vp]
             b.ti_tanh_norm_rows.argtypes = [_vp, _vp, _i, _i, _f, _vp, _vp, _vp, _i, _vp, _i, _vp]
             b.ti_tanh_norm_pair.argtypes = [_vp, _i, _i, _f, _vp, _vp, _vp, _i, _f, _vp, _vp, _vp, _i, _vp]
+            b.ti_layer_norm_rows.argtypes = [_vp, _vp, _vp, _vp, _i, _i, _f, _vp, _i, _vp]
+            b.ti_norm_sum_rows.argtypes = [_vp, _vp, _vp, _vp, _f, _f, _vp, _i, _i, _i, _vp, _vp, _f, _vp, _i, _vp]
+            b.ti_unary_rows.argtypes = [_vp, _ll, _i, _vp, _i, _vp]
             b.ti_cap_rows.argtypes = [_vp, _ll, _f, _vp]
             b.ti_add_row.argtypes = [_vp, _i, _vp, _i, _i, _vp]
             b.ti_depth_mix.argtypes = [_vp, _vp, _ll, _i, _vp, _vp]
@@ -227,9 +234,13 @@ class StateOps:
 
     # ---- sums that pass a gate ---------------------------------------------------------------------
     def gated_add(self, y, target):
-        """``x += scale * sigmoid(gate + bias) * y`` for a ``parts.base.GatedSum`` ``target``."""
+        """``x += scale * sigmoid(gate + bias) * y`` (or, without a gate, ``x += scale * y``) for a
+        ``parts.base.GatedSum`` ``target``."""
         self.flush()
         x, gate, bias = target.x, target.gate, target.bias
+        if gate is None:
+            self.add_scaled(x, y, target.scale)
+            return
         for v in (x, gate, y):
             self._want(v.dtype == torch.float32 and v.stride(1) == 1 and tuple(v.shape) == tuple(x.shape),
                        "gated_add: float32 rows of one shape")
@@ -295,6 +306,44 @@ class StateOps:
             y.data_ptr(), y.shape[0], n, float(alpha1), weight1.data_ptr(), _ptr(bias1), residual.data_ptr(),
             residual.stride(0), float(alpha2), weight2.data_ptr(), _ptr(bias2), out.data_ptr(), _CODE[out.dtype],
             self._stream()))
+
+    def layer_norm(self, x, weight, bias, eps, out, rows=None):
+        """``(x - mean) / sqrt(var + eps) * weight + bias`` for every row of the float32 ``x`` (of the rows ``rows`` if
+        given), ``var`` the mean of the squared deviations."""
+        n = x.shape[1]
+        num = x.shape[0] if rows is None else rows.shape[0]
+        self._want(x.dtype == torch.float32 and x.is_contiguous() and out.is_contiguous() and tuple(out.shape) == (num, n)
+                   and (rows is None or rows.dtype == torch.int32), "layer_norm: contiguous float32 rows, rows of the same length out")
+        for v in (weight, bias):
+            self._want(v.dtype == torch.float32 and v.is_contiguous() and v.shape[0] == n,
+                       "layer_norm: a float32 weight and bias per element")
+        self._rw(self.rows_lib.ti_layer_norm_rows(x.data_ptr(), weight.data_ptr(), bias.data_ptr(), _ptr(rows), num, n,
+                                                  float(eps), out.data_ptr(), _CODE[out.dtype], self._stream()))
+
+    def norm_sum(self, a, b, weight_a, weight_b, eps, residual, scale, then=None):
+        """``residual += scale * (rms(a) * weight_a + rms(b) * weight_b)``, every row of ``a`` and ``b`` over the root of its
+        mean square (+ ``eps``).  ``then = (weight, bias, eps, out)``: ``out`` gets the layer norm of the new rows in the
+        same launch."""
+        t, n = a.shape
+        for v in (a, b):
+            self._want(v.dtype == torch.float32 and v.is_contiguous() and tuple(v.shape) == (t, n), "norm_sum: float32 rows of one shape")
+        for v in (weight_a, weight_b, *(then[:2] if then is not None else ())):
+            self._want(v.dtype == torch.float32 and v.is_contiguous() and v.shape[0] == n, "norm_sum: a float32 weight per element")
+        self._want(residual.dtype == torch.float32 and residual.stride(1) == 1 and tuple(residual.shape) == (t, n),
+                   "norm_sum: a float32 residual of the rows' shape")
+        w2, b2, eps2, out = then if then is not None else (None, None, 0.0, None)
+        self._want(out is None or (out.is_contiguous() and tuple(out.shape) == (t, n)), "norm_sum: the normed rows out")
+        self._rw(self.rows_lib.ti_norm_sum_rows(
+            a.data_ptr(), b.data_ptr(), weight_a.data_ptr(), weight_b.data_ptr(), float(eps), float(scale),
+            residual.data_ptr(), residual.stride(0), t, n, _ptr(w2), _ptr(b2), float(eps2), _ptr(out),
+            _CODE[out.dtype] if out is not None else 0, self._stream()))
+
+    def unary_rows(self, x, kind, out):
+        """``out = act(x)`` element by element over a contiguous float32 tensor; ``kind`` "relu2": the square of relu."""
+        self._want(x.dtype == torch.float32 and x.is_contiguous() and out.is_contiguous() and out.shape == x.shape,
+                   "unary_rows: contiguous float32 in, the same shape out")
+        self._rw(self.rows_lib.ti_unary_rows(x.data_ptr(), x.numel(), UNARY_KINDS[kind], out.data_ptr(), _CODE[out.dtype],
+                                             self._stream()))
 
     def cap_rows(self, x, cap):
         """``x = cap tanh(x / cap)`` over a contiguous float32 tensor, in place."""

@@ -91,11 +91,11 @@ class CompositeSpec:
 class GatedSum:
     """Where a sublayer's last product lands when its result passes a gate on the way into the
     residual stream: ``x += scale * sigmoid(gate + bias) * result``, element by element.  ``gate`` is
-    float32 ``[T, width]``, ``bias`` float32 ``[width]``.  ``ops.linear(a, w, target, accumulate=True)``
-    takes it in the place of a float32 residual."""
+    float32 ``[T, width]``, ``bias`` float32 ``[width]``; both None: ``x += scale * result``.
+    ``ops.linear(a, w, target, accumulate=True)`` takes it in the place of a float32 residual."""
     x: torch.Tensor
-    gate: torch.Tensor
-    bias: torch.Tensor
+    gate: Optional[torch.Tensor]
+    bias: Optional[torch.Tensor]
     scale: float
 
     @property
@@ -108,6 +108,9 @@ class Part:
     # a mixer or feed-forward that touches its residual by one closing ``ops.linear(..., accumulate=True)``
     # alone: a block may then hand it a ``GatedSum``
     ends_in_linear = False
+    # a mixer or feed-forward that takes a ``GatedSum`` without a gate (a factor on what it adds) in the
+    # place of its residual, besides those that end in a product
+    takes_factor = False
 
     def weight_specs(self) -> dict[str, WeightSpec]:
         return {}
@@ -123,6 +126,35 @@ class Part:
     def shared_weights(self) -> dict[str, torch.Tensor]:
         """Tensors another part may alias (for instance the embedding table for a tied head)."""
         return {}
+
+
+def residual_and_factor(target) -> "tuple[torch.Tensor, float]":
+    """The float32 residual behind a sublayer's target and the factor on what is added to it."""
+    if isinstance(target, torch.Tensor):
+        return target, 1.0
+    if target.gate is not None:
+        raise ValueError("this part adds to its residual with a factor, not through a gate")
+    return target.x, target.scale
+
+
+class ProjectedMixer(Part):
+    """A mixer that is one product of its input, something in between, and one product into its residual:
+    ``residual += w_o mix(w_in h)``.  ``mix(ops, proj, step, cache, dtype)`` gets the float32 columns of the
+    first product (a column slice of a wider one is fine) and returns the rows that the last one reads, so a
+    part that holds several such mixers can run their products as one."""
+    category = "mixer"
+    ends_in_linear = True
+    defers = False            # the closing product may be held back for what follows (``ops.linear``)
+    w_in = w_o = None
+
+    def mix(self, ops, proj, step, cache, dtype):
+        raise NotImplementedError
+
+    def forward(self, ops, h, residual, step, cache):
+        proj = torch.empty((h.shape[0], self.w_in.shape[0]), dtype=torch.float32, device=h.device)
+        ops.linear(h, self.w_in, proj)
+        out = self.mix(ops, proj, step, cache, h.dtype)
+        ops.linear(out, self.w_o, residual, accumulate=True, may_defer=self.defers)
 
 
 _REGISTRY: dict[tuple[str, str], Callable[..., Part]] = {}
@@ -149,3 +181,14 @@ def build_part(category: str, spec: PartSpec, **extra: Any) -> Part:
 def as_float32(t: torch.Tensor) -> torch.Tensor:
     """Norm weights and tables are used in float32; widening bfloat16 is exact."""
     return t if t.dtype == torch.float32 else t.to(torch.float32)
+
+
+def stack_rows(mats, width: int) -> torch.Tensor:
+    """The matrices one below the other (widened if their storage differs), with zero rows up to
+    a multiple of 16 that the tensor-core products take."""
+    if len({m.dtype for m in mats}) > 1:
+        mats = [m.to(torch.float32) for m in mats]
+    rows = sum(m.shape[0] for m in mats)
+    if rows % 16:
+        mats = list(mats) + [torch.zeros((16 - rows % 16, width), dtype=mats[0].dtype, device=mats[0].device)]
+    return torch.cat(mats, dim=0)

@@ -10,6 +10,8 @@ mixer's and the feed-forward's last product.  A layer without a feed-forward sto
 residual stream, ``x += m sigmoid(Wg h + bg) * sublayer(h)``, with an optional shift of the mixer's
 input towards the token before.
 
+``scaled_prenorm``: ``prenorm`` with a constant factor on what each sublayer adds, ``x += m * sublayer(norm(x))``.
+
 ``sandwich``: a norm before and behind each sublayer, ``x += norm1b(mixer(norm1(x)))`` then
 ``x += norm2b(ffn(norm2(x)))``.
 
@@ -23,6 +25,7 @@ import torch
 
 from .base import (MATRIX, NORM_WEIGHT, NORM_ZERO, CompositeSpec, FixedStateSpec, GatedSum, Part, WeightSpec, as_float32,
                    register_part)
+from .norm import LayerNorm
 
 
 class PreNormBlock(Part):
@@ -104,6 +107,39 @@ class GatedPreNormBlock(Part):
         if self.ffn is not None:
             h = self.ffn_norm.forward(ops, x, step.act_dtype)
             self._add(ops, self.ffn, lambda y: self.ffn.forward(ops, h, y, step), h, x, self.gates[1])
+
+
+class ScaledPreNormBlock(PreNormBlock):
+    """Pre-norm with a constant factor on what each sublayer adds: ``x += m mixer(norm1(x))``, then, where the
+    layer has one, ``x += m ffn(norm2(x))`` with ``m`` = ``multiplier``.  The factor travels with the residual (a
+    ``GatedSum`` without a gate) into the sublayer's last kernel; a part that does not take one writes into
+    rows of its own, which are then added.  A mixer that can norm the residual behind its own sum
+    (``forward_then``) hands the feed-forward its input."""
+
+    def __init__(self, mixer, mixer_norm, ffn=None, ffn_norm=None, multiplier: float = 1.0):
+        super().__init__(mixer, mixer_norm, ffn, ffn_norm)
+        self.multiplier = float(multiplier)
+
+    def _add(self, ops, part, run, x):
+        if self.multiplier == 1.0:
+            return run(x)
+        if part.ends_in_linear or part.takes_factor:
+            return run(GatedSum(x, None, None, self.multiplier))
+        y = torch.zeros_like(x)
+        run(y)
+        ops.flush()
+        ops.add_scaled(x, y, self.multiplier)
+
+    def forward(self, ops, x, step, cache):
+        h = self.mixer_norm.forward(ops, x, step.act_dtype)
+        if self.ffn is not None and self.mixer.takes_factor and hasattr(self.mixer, "forward_then") and isinstance(self.ffn_norm, LayerNorm):
+            h = self._add(ops, self.mixer, lambda y: self.mixer.forward_then(ops, h, y, step, cache, self.ffn_norm), x)
+        else:
+            self._add(ops, self.mixer, lambda y: self.mixer.forward(ops, h, y, step, cache), x)
+            if self.ffn is not None:
+                h = self.ffn_norm.forward(ops, x, step.act_dtype)
+        if self.ffn is not None:
+            self._add(ops, self.ffn, lambda y: self.ffn.forward(ops, h, y, step), x)
 
 
 class ParallelBlock(Part):
@@ -233,6 +269,7 @@ class OutputNormBlock(Part):
 
 register_part("block", "prenorm", PreNormBlock)
 register_part("block", "gated_prenorm", GatedPreNormBlock)
+register_part("block", "scaled_prenorm", ScaledPreNormBlock)
 register_part("block", "output_norm", OutputNormBlock)
 register_part("block", "sandwich", SandwichBlock)
 register_part("block", "parallel", ParallelBlock)

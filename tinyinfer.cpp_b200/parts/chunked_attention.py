@@ -17,6 +17,13 @@ For token ``i`` and query head ``a`` (kv head ``a // (heads / kv_heads)``):
 query and key head by itself with one weight of ``head_dim`` elements, so other designs can use the
 part: with everything off it is plain causal grouped-query attention with a query/key norm.
 
+More options, for heads that are prepared one by one (``heads_prepare_store``): ``norm_before`` False leaves the
+norm in front of the turn out (no ``q.norm``, ``k.norm``); ``norm_after`` divides every query and key head by its
+root mean square behind the turn; ``bias`` adds a stored bias to q, k and v (``q.b`` ...); ``query_factor = (coef,
+every)`` multiplies the query at position ``p`` by ``1 + coef ln(floor((p + 1) / every) + 1)``; ``values_from_keys``
+takes the projected keys, before norm and turn, as values (no ``v``); ``sink`` adds ``exp(sink[a])`` to the
+softmax's denominator (a number per head, without a key or a value).
+
 ``value_mix`` ties the values of several layers together: the layer with ``"source"`` leaves its values
 ``v1`` (float32, in the step's scratch), and a later layer with ``"mix"`` caches ``(1 - l) v + l v1`` of
 the same token (``l`` the number in the tensor ``vmix``).
@@ -28,18 +35,19 @@ from typing import Optional
 import torch
 
 from ..config.plan import PartSpec
-from .base import MATRIX, NORM_WEIGHT, NORM_ZERO, PagedKVSpec, Part, WeightSpec, as_float32, build_part, register_part
+from .base import (MATRIX, NORM_WEIGHT, NORM_ZERO, PagedKVSpec, ProjectedMixer, WeightSpec, as_float32, build_part,
+                   register_part, stack_rows)
 
 
-class ChunkedAttention(Part):
-    category = "mixer"
-    ends_in_linear = True
+class ChunkedAttention(ProjectedMixer):
+    defers = True
 
     def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, head_dim: int, v_head_dim: int,
                  scale: float, qk_norm_eps: float, position: PartSpec, chunk: Optional[int] = None,
                  window: Optional[int] = None, softcap: Optional[float] = None,
                  head_temperature: bool = True, head_gate: bool = True, norm_per_head: bool = False,
-                 value_mix: Optional[str] = None):
+                 value_mix: Optional[str] = None, norm_before: bool = True, norm_after: bool = False, bias: bool = False,
+                 query_factor=None, values_from_keys: bool = False, sink: bool = False):
         if value_mix not in (None, "source", "mix"):
             raise ValueError(f"value_mix must be None, 'source' or 'mix', got {value_mix!r}")
         if num_heads % num_kv_heads:
@@ -60,18 +68,39 @@ class ChunkedAttention(Part):
         self.norm_per_head = bool(norm_per_head)
         if self.norm_per_head and value_mix is not None:
             raise ValueError("values are mixed beside a norm over whole rows only")
+        self.norm_before, self.norm_after, self.has_bias = bool(norm_before), bool(norm_after), bool(bias)
+        self.query_factor = None if query_factor is None else (float(query_factor[0]), int(query_factor[1]))
+        self.values_from_keys, self.has_sink = bool(values_from_keys), bool(sink)
+        # heads one by one, with whatever of these options there is
+        self.by_heads = (not self.norm_before or self.norm_after or self.has_bias or self.query_factor is not None
+                         or self.values_from_keys)
+        if self.by_heads and (value_mix is not None or (self.norm_before and not self.norm_per_head)):
+            raise ValueError("heads that are prepared one by one have norms per head and values of their own")
+        if self.values_from_keys and head_dim != v_head_dim:
+            raise ValueError(f"values of {v_head_dim} elements cannot be keys of {head_dim}")
+        if self.query_factor is not None and self.query_factor[1] < 1:
+            raise ValueError(f"the query's factor grows every {query_factor[1]} positions; that must be positive")
         self.position = build_part("position", position)
         self.value_mix, self.mix_share = value_mix, 0.0
         self.nq, self.nk = self.num_heads * self.head_dim, self.num_kv_heads * self.head_dim
-        self.nv, self.no = self.num_kv_heads * self.v_head_dim, self.num_heads * self.v_head_dim
-        self.w_in = self.w_o = self.q_norm = self.k_norm = self.temp = None
+        self.nv = 0 if self.values_from_keys else self.num_kv_heads * self.v_head_dim
+        self.no = self.num_heads * self.v_head_dim
+        self.projected = ("q", "k") if self.values_from_keys else ("q", "k", "v")
+        self.q_norm = self.k_norm = self.temp = self.sink = self.bias = None
 
     def weight_specs(self):
         h = self.hidden_size
-        specs = {"q": WeightSpec((self.nq, h), MATRIX), "k": WeightSpec((self.nk, h), MATRIX),
-                 "v": WeightSpec((self.nv, h), MATRIX), "o": WeightSpec((h, self.no), MATRIX),
-                 "q.norm": WeightSpec((self.head_dim if self.norm_per_head else self.nq,), NORM_WEIGHT),
-                 "k.norm": WeightSpec((self.head_dim if self.norm_per_head else self.nk,), NORM_WEIGHT)}
+        rows = {"q": self.nq, "k": self.nk, "v": self.nv}
+        specs = {"o": WeightSpec((h, self.no), MATRIX)}
+        for name in self.projected:
+            specs[name] = WeightSpec((rows[name], h), MATRIX)
+            if self.has_bias:
+                specs[name + ".b"] = WeightSpec((rows[name],), NORM_ZERO)
+        if self.norm_before:
+            specs["q.norm"] = WeightSpec((self.head_dim if self.norm_per_head else self.nq,), NORM_WEIGHT)
+            specs["k.norm"] = WeightSpec((self.head_dim if self.norm_per_head else self.nk,), NORM_WEIGHT)
+        if self.has_sink:
+            specs["sink"] = WeightSpec((self.num_heads,), NORM_ZERO)
         if self.value_mix is not None:                # the source may store a number that it does not use
             specs["vmix"] = WeightSpec((), NORM_ZERO, optional=self.value_mix == "source")
         if self.head_temperature:
@@ -81,13 +110,15 @@ class ChunkedAttention(Part):
         return specs
 
     def load_weights(self, tensors, ops):
-        mats = [tensors[n] for n in (("q", "k", "v", "g") if self.head_gate else ("q", "k", "v"))]
-        if len({m.dtype for m in mats}) > 1:          # mixed storage: widen, never narrow
-            mats = [m.to(torch.float32) for m in mats]
-        self.w_in = ops.pack_linear(torch.cat(mats, dim=0))
+        mats = [tensors[n] for n in self.projected + (("g",) if self.head_gate else ())]
+        self.w_in = ops.pack_linear(stack_rows(mats, self.hidden_size))
         self.w_o = ops.pack_linear(tensors["o"])
-        self.q_norm = as_float32(tensors["q.norm"]).contiguous()
-        self.k_norm = as_float32(tensors["k.norm"]).contiguous()
+        if self.norm_before:
+            self.q_norm = as_float32(tensors["q.norm"]).contiguous()
+            self.k_norm = as_float32(tensors["k.norm"]).contiguous()
+        if self.has_bias:
+            self.bias = torch.cat([as_float32(tensors[n + ".b"]) for n in self.projected]).contiguous()
+        self.sink = as_float32(tensors["sink"]).contiguous() if self.has_sink else None
         self.temp = as_float32(tensors["temp"]).contiguous() if self.head_temperature else None
         if self.value_mix == "mix":                   # a constant of the model
             self.mix_share = float(as_float32(tensors["vmix"]).reshape(()).item())
@@ -98,15 +129,19 @@ class ChunkedAttention(Part):
         return PagedKVSpec(self.num_kv_heads, self.head_dim, self.window,
                            None if self.v_head_dim == self.head_dim else self.v_head_dim, 0, self.chunk)
 
-    def forward(self, ops, h, residual, step, cache):
-        t = h.shape[0]
-        proj = torch.empty((t, self.w_in.shape[0]), dtype=torch.float32, device=h.device)
-        ops.linear(h, self.w_in, proj)
-        q = torch.empty((t, self.nq), dtype=h.dtype, device=h.device)
-        rotation = self.position.rotation(h.device)
+    def mix(self, ops, proj, step, cache, dtype):
+        t, dev = proj.shape[0], proj.device
+        q = torch.empty((t, self.nq), dtype=dtype, device=dev)
+        rotation = self.position.rotation(dev)
         if self.value_mix == "source":
             step.scratch["value_mix"] = proj[:, self.nq + self.nk:self.nq + self.nk + self.nv]
-        if rotation.kind == "neox" or self.value_mix is not None:
+        if self.by_heads:
+            ops.heads_prepare_store(proj, rotation, step, cache, q, self.num_heads, self.num_kv_heads, self.head_dim,
+                                    self.v_head_dim, bias=self.bias,
+                                    pre_norm=(self.q_norm, self.k_norm, self.eps) if self.norm_before else None,
+                                    post_norm_eps=self.eps if self.norm_after else None, query_factor=self.query_factor,
+                                    values_from_keys=self.values_from_keys)
+        elif rotation.kind == "neox" or self.value_mix is not None:
             mixed = (step.scratch["value_mix"], self.mix_share) if self.value_mix == "mix" else None
             ops.qkv_turn_store(proj, rotation, None, step, cache, q, self.num_heads, self.num_kv_heads, self.head_dim,
                                self.v_head_dim, row_norm=(self.q_norm, self.k_norm, self.eps), value_mix=mixed)
@@ -114,12 +149,13 @@ class ChunkedAttention(Part):
             ops.qk_rownorm_rope_store(proj, self.q_norm, self.k_norm, self.eps, rotation, step, cache, q,
                                       self.num_heads, self.num_kv_heads, self.head_dim, self.v_head_dim,
                                       per_head=self.norm_per_head)
-        gate = proj[:, self.nq + self.nk + self.nv:] if self.head_gate else None
-        out = torch.empty((t, self.no), dtype=h.dtype, device=h.device)
+        at_g = self.nq + self.nk + self.nv
+        gate = proj[:, at_g:at_g + self.num_heads] if self.head_gate else None
+        out = torch.empty((t, self.no), dtype=dtype, device=dev)
         ops.attention_options(q, step, cache, out, self.num_heads, self.num_kv_heads, self.head_dim,
                               self.v_head_dim, self.scale, window=self.window, chunk=self.chunk,
-                              softcap=self.softcap, head_scale=self.temp, gate=gate, gate_per_head=True)
-        ops.linear(out, self.w_o, residual, accumulate=True, may_defer=True)
+                              softcap=self.softcap, head_scale=self.temp, sink=self.sink, gate=gate, gate_per_head=True)
+        return out
 
 
 register_part("mixer", "chunked_attention", ChunkedAttention)

@@ -20,14 +20,10 @@ from __future__ import annotations
 
 import torch
 
-from .base import MATRIX, NORM_WEIGHT, NORM_ZERO, FixedStateSpec, Part, WeightSpec, as_float32, register_part
-from .state_mixers import _stack_rows
+from .base import MATRIX, NORM_ZERO, FixedStateSpec, ProjectedMixer, WeightSpec, as_float32, register_part, stack_rows
 
 
-class GatedLinearRecurrence(Part):
-    category = "mixer"
-    ends_in_linear = True
-
+class GatedLinearRecurrence(ProjectedMixer):
     def __init__(self, hidden_size: int, width: int, blocks: int, conv_taps: int, decay_power: float = 8.0):
         self.hidden_size, self.width, self.blocks = int(hidden_size), int(width), int(blocks)
         self.conv_taps, self.decay_power = int(conv_taps), float(decay_power)
@@ -35,7 +31,7 @@ class GatedLinearRecurrence(Part):
             raise ValueError(f"{self.width} channels do not fall into {self.blocks} equal blocks")
         if self.conv_taps < 1:
             raise ValueError(f"the short convolution needs at least one tap, got {conv_taps}")
-        self.w_in = self.w_o = self.w_gates = self.conv_w = self.conv_b = None
+        self.w_gates = self.conv_w = self.conv_b = None
         self.y_bias = self.x_bias = self.gate_bias = self.log_decay = None
 
     def weight_specs(self):
@@ -49,7 +45,7 @@ class GatedLinearRecurrence(Part):
                 "lam": WeightSpec((n,), NORM_ZERO), "o": WeightSpec((h, n), MATRIX)}
 
     def load_weights(self, tensors, ops):
-        self.w_in = ops.pack_linear(_stack_rows([tensors["y"], tensors["x"]], self.hidden_size))
+        self.w_in = ops.pack_linear(stack_rows([tensors["y"], tensors["x"]], self.hidden_size))
         self.w_o = ops.pack_linear(tensors["o"])
         ra, ri = tensors["ra"], tensors["ri"]
         if ra.dtype != ri.dtype:                      # mixed storage: widen, never narrow
@@ -66,15 +62,13 @@ class GatedLinearRecurrence(Part):
     def cache_spec(self):
         return FixedStateSpec((self.width * self.conv_taps,), torch.float32)      # the state, taps - 1 rows
 
-    def forward(self, ops, h, residual, step, cache):
-        t, dev, n = h.shape[0], h.device, self.width
-        proj = torch.empty((t, self.w_in.shape[0]), dtype=torch.float32, device=dev)
-        ops.linear(h, self.w_in, proj)
+    def mix(self, ops, proj, step, cache, dtype):
+        t, dev, n = proj.shape[0], proj.device, self.width
         u = torch.empty((t, n), dtype=torch.float32, device=dev)
         ops.causal_conv(proj[:, n:2 * n], self.conv_w, step, cache, n, u, renew=True, in_bias=self.x_bias, bias=self.conv_b)
-        out = torch.empty((t, n), dtype=h.dtype, device=dev)
+        out = torch.empty((t, n), dtype=dtype, device=dev)
         ops.gated_recurrence(u, self.w_gates, self.gate_bias, self.log_decay, proj[:, :n], self.y_bias, step, cache, out)
-        ops.linear(out, self.w_o, residual, accumulate=True)
+        return out
 
 
 register_part("mixer", "gated_linear_recurrence", GatedLinearRecurrence)

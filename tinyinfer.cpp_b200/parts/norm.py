@@ -101,6 +101,36 @@ class GroupRMSNorm(Part):
 register_part("norm", "group_rmsnorm", GroupRMSNorm)
 
 
+class LayerNorm(Part):
+    """``(x - mean) / sqrt(var + eps) * w + b`` with a weight and a bias per element (tensors ``<tensor>`` and
+    ``<tensor>.b``); ``var`` is the mean of the squared deviations."""
+    category = "norm"
+
+    def __init__(self, size: int, eps: float, tensor: str = "weight"):
+        self.size, self.eps, self.tensor = int(size), float(eps), str(tensor)
+        self.weight = self.bias = None
+
+    def weight_specs(self):
+        return {self.tensor: WeightSpec((self.size,), NORM_WEIGHT), self.tensor + ".b": WeightSpec((self.size,), NORM_ZERO)}
+
+    def load_weights(self, tensors, ops):
+        self.weight = as_float32(tensors[self.tensor]).contiguous()
+        self.bias = as_float32(tensors[self.tensor + ".b"]).contiguous()
+
+    def forward(self, ops, x: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
+        out = torch.empty((x.shape[0], self.size), dtype=out_dtype, device=x.device)
+        ops.layer_norm(x, self.weight, self.bias, self.eps, out)
+        return out
+
+    def forward_rows(self, ops, x: torch.Tensor, rows: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
+        out = torch.empty((rows.shape[0], self.size), dtype=out_dtype, device=x.device)
+        ops.layer_norm(x, self.weight, self.bias, self.eps, out, rows=rows)
+        return out
+
+
+register_part("norm", "layer_norm", LayerNorm)
+
+
 class DynamicTanh(Part):
     """A norm that takes no mean and no variance: ``tanh(alpha * x) * w + b`` with one scalar
     ``alpha``, a weight and a bias per element (tensors ``<tensor>``, ``<tensor>.alpha``,

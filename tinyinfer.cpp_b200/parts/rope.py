@@ -22,6 +22,7 @@ Kinds built in:
 
 ``rope_stretched`` (YaRN) answers with either pairing: frequencies that turn fast stay, slow ones are
 divided by ``factor``, a ramp lies between; and ``Rotation.scale`` multiplies both sine and cosine.
+``rope_wavelength`` (Llama 3.1) divides by the wavelength instead, without a factor on sine and cosine.
 
 ``inv_freq`` is computed once on the host in double precision and rounded to float32; the
 angle, its sine and cosine are float32 on the device.
@@ -126,6 +127,43 @@ class RopeStretched(RopeNeox):
         return Rotation(self.layout, self.rotary_dim, _TABLES[key], scale=0.1 * math.log(self.factor) + 1.0)
 
 
+class RopeWavelength(RopeNeox):
+    """Frequencies scaled by their wavelength ``l = 2 pi / f`` (the scaling of Llama 3.1): ``f`` stays where ``l <
+    original / high``, becomes ``f / factor`` where ``l > original / low``, and ``(1 - s) f / factor + s f`` with ``s =
+    (original / l - low) / (high - low)`` between the two.  ``layout``: ``neox`` or ``interleaved``."""
+
+    def __init__(self, head_dim: int, theta: float, factor: float, original: float, low: float, high: float,
+                 rotary_dim: Optional[int] = None, layout: str = "neox"):
+        super().__init__(head_dim, theta, rotary_dim)
+        if layout not in ("interleaved", "neox"):
+            raise ValueError(f"pairing {layout!r}; known: interleaved, neox")
+        self.factor, self.original = float(factor), float(original)
+        self.low, self.high, self.layout = float(low), float(high), layout
+        if not (self.factor > 0 and self.original > 0 and self.low > 0 and self.high > 0 and self.theta > 0):
+            raise ValueError("frequencies scaled by wavelength need positive constants")
+
+    def inv_freq(self) -> torch.Tensor:
+        import math
+        out = []
+        for k in range(self.rotary_dim // 2):
+            f = self.theta ** (-2.0 * k / self.rotary_dim)
+            wave = 2.0 * math.pi / f
+            if wave < self.original / self.high:
+                out.append(f)
+            elif wave > self.original / self.low:
+                out.append(f / self.factor)
+            else:                                     # low < high here, or the bounds meet in this wavelength
+                s = (self.original / wave - self.low) / (self.high - self.low) if self.high != self.low else 1.0
+                out.append((1.0 - s) * f / self.factor + s * f)
+        return torch.tensor(out, dtype=torch.float64).to(torch.float32)
+
+    def rotation(self, device) -> Rotation:
+        key = ("wavelength", self.rotary_dim, self.theta, self.factor, self.original, self.low, self.high, str(device))
+        if key not in _TABLES:
+            _TABLES[key] = self.inv_freq().to(device)
+        return Rotation(self.layout, self.rotary_dim, _TABLES[key])
+
+
 class NoPosition(Part):
     """Heads are normed and stored without a rotation."""
     category = "position"
@@ -140,4 +178,5 @@ class NoPosition(Part):
 register_part("position", "rope_neox", RopeNeox)
 register_part("position", "rope_interleaved", RopeInterleaved)
 register_part("position", "rope_stretched", RopeStretched)
+register_part("position", "rope_wavelength", RopeWavelength)
 register_part("position", "none", NoPosition)

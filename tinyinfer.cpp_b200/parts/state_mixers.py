@@ -43,18 +43,8 @@ from __future__ import annotations
 
 import torch
 
-from .base import MATRIX, NORM_WEIGHT, NORM_ZERO, FixedStateSpec, Part, WeightSpec, as_float32, register_part
-
-
-def _stack_rows(mats, width):
-    """The matrices one below the other (widened if their storage differs), with zero rows up to
-    a multiple of 16 that the tensor-core products take."""
-    if len({m.dtype for m in mats}) > 1:
-        mats = [m.to(torch.float32) for m in mats]
-    rows = sum(m.shape[0] for m in mats)
-    if rows % 16:
-        mats = list(mats) + [torch.zeros((16 - rows % 16, width), dtype=mats[0].dtype, device=mats[0].device)]
-    return torch.cat(mats, dim=0)
+from .base import (MATRIX, NORM_WEIGHT, NORM_ZERO, FixedStateSpec, Part, ProjectedMixer, WeightSpec, as_float32,
+                   register_part, stack_rows)
 
 
 class GatedDeltaMixer(Part):
@@ -87,7 +77,7 @@ class GatedDeltaMixer(Part):
 
     def load_weights(self, tensors, ops):
         # columns of the product: q, k, v (what the convolution reads), the gate, beta's logit, the decay's argument
-        self.w_in = ops.pack_linear(_stack_rows([tensors[n] for n in ("q", "k", "v", "g", "b", "a")], self.hidden_size))
+        self.w_in = ops.pack_linear(stack_rows([tensors[n] for n in ("q", "k", "v", "g", "b", "a")], self.hidden_size))
         self.conv_w = torch.cat([as_float32(tensors[n + ".conv"]) for n in ("q", "k", "v")], dim=0).contiguous()
         self.a_log = as_float32(tensors["A_log"]).contiguous()
         self.dt_bias = as_float32(tensors["dt_bias"]).contiguous()
@@ -134,7 +124,7 @@ class MatrixMemoryMixer(Part):
                 "norm": WeightSpec((self.nv,), NORM_WEIGHT), "o": WeightSpec((h, self.nv), MATRIX)}
 
     def load_weights(self, tensors, ops):
-        self.w_in = ops.pack_linear(_stack_rows([tensors[n] for n in ("q", "k", "v", "g", "i", "f")], self.hidden_size))
+        self.w_in = ops.pack_linear(stack_rows([tensors[n] for n in ("q", "k", "v", "g", "i", "f")], self.hidden_size))
         self.bias_i = as_float32(tensors["i.b"]).contiguous()
         self.bias_f = as_float32(tensors["f.b"]).contiguous()
         self.norm = as_float32(tensors["norm"]).contiguous()
@@ -160,10 +150,7 @@ class MatrixMemoryMixer(Part):
         ops.linear(out, self.w_o, residual, accumulate=True)
 
 
-class GatedLinearAttention(Part):
-    category = "mixer"
-    ends_in_linear = True
-
+class GatedLinearAttention(ProjectedMixer):
     def __init__(self, hidden_size: int, num_heads: int, head_dim: int, v_head_dim: int, tau: float, norm_eps: float,
                  decay_rank=None):
         self.hidden_size, self.num_heads = int(hidden_size), int(num_heads)
@@ -174,7 +161,7 @@ class GatedLinearAttention(Part):
         # inner width of the decay's products: the stored tensors' own unless given (random weights need it)
         self.decay_rank = None if decay_rank is None else int(decay_rank)
         self.nk, self.nv = self.num_heads * self.head_dim, self.num_heads * self.v_head_dim
-        self.w_in = self.w_o = self.a2 = self.a2_bias = self.norm = None
+        self.a2 = self.a2_bias = self.norm = None
         self.rank = 0
 
     def weight_specs(self):
@@ -187,7 +174,7 @@ class GatedLinearAttention(Part):
 
     def load_weights(self, tensors, ops):
         # columns of the product: q, k, v, the gate, the decay's inner row
-        self.w_in = ops.pack_linear(_stack_rows([tensors[n] for n in ("q", "k", "v", "g", "a1")], self.hidden_size))
+        self.w_in = ops.pack_linear(stack_rows([tensors[n] for n in ("q", "k", "v", "g", "a1")], self.hidden_size))
         self.rank = tensors["a1"].shape[0]
         self.a2 = ops.pack_linear(tensors["a2"])
         if self.a2.shape[1] != self.rank:
@@ -199,19 +186,17 @@ class GatedLinearAttention(Part):
     def cache_spec(self):
         return FixedStateSpec((self.nk * self.v_head_dim,), torch.float32)
 
-    def forward(self, ops, h, residual, step, cache):
-        t, dev, nk, nv = h.shape[0], h.device, self.nk, self.nv
-        proj = torch.empty((t, self.w_in.shape[0]), dtype=torch.float32, device=dev)
-        ops.linear(h, self.w_in, proj)
+    def mix(self, ops, proj, step, cache, dtype):
+        t, dev, nk, nv = proj.shape[0], proj.device, self.nk, self.nv
         at_g, at_a = 2 * nk + nv, 2 * nk + 2 * nv
         decay = torch.empty((t, nk), dtype=torch.float32, device=dev)
         ops.low_rank_decay(proj[:, at_a:at_a + self.rank], self.a2, self.a2_bias, self.tau, decay)
-        out = torch.empty((t, nv), dtype=h.dtype, device=dev)
+        out = torch.empty((t, nv), dtype=dtype, device=dev)
         ops.matrix_state("decayed_sum", proj[:, :nk], proj[:, nk:2 * nk], proj[:, 2 * nk:at_g], None, None, None, None,
                          step, cache, out, heads=self.num_heads, kv_heads=self.num_heads, dk=self.head_dim,
                          dv=self.v_head_dim, eps=self.eps, norm_weight=self.norm, gate=proj[:, at_g:at_a],
                          gate_act="silu", decay=decay)
-        ops.linear(out, self.w_o, residual, accumulate=True)
+        return out
 
 
 register_part("mixer", "gated_linear_attention", GatedLinearAttention)
