@@ -1276,6 +1276,198 @@ def vametar_arm(args) -> int:
     return 0
 
 
+# ---- the Saberax decoder beside the Feruzen decoder at equal sizes ------------------------------
+# (width, heads, kv heads, head size, window, chunk, channels and blocks of the linear recurrence, taps, heads of the
+#  linear attention with their key and value size, inner width of its decay, dense ff, experts, top, expert ff, groups
+#  (count, keep), shared ff, blocks of [window attention beside linear attention + dense, causal attention beside the
+#  recurrence + experts, chunked attention + experts] layers)
+SABERAX_SIZES = {
+    "w1024": (1024, 16, 4, 64, 1024, 2048, 1024, 8, 4, 8, 64, 128, 16, 2816, 16, 2, 704, (4, 2), 704, 2),
+    "w2048": (2048, 16, 4, 128, 1024, 2048, 2048, 8, 4, 16, 128, 128, 16, 5632, 32, 4, 1408, (4, 2), 1408, 2),
+    "w4096": (4096, 32, 8, 128, 1024, 2048, 4096, 16, 4, 32, 128, 128, 16, 11008, 64, 4, 1408, (8, 4), 2816, 1),
+}
+
+
+def saberax_config(size):
+    w, h, g, d, window, chunk, rw, rb, taps, lh, ld, lv, rank, ff, experts, top, eff, groups, sff, blocks = size
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "router": {"experts": experts, "top": top, "scale": 2.0, "groups": {"count": groups[0], "keep": groups[1]}},
+           "expert": {"ff": eff}, "shared": {"ff": sff}}
+    heads = {"heads": h, "kv_heads": g, "dim": d, "vdim": d, "scale": d ** -0.5}
+    layers = [
+        {"type": "parallel_2", "mlp": dense, "mixer": {
+            "left": dict(heads, mask={"size": window}, rot={"dims": d // 2, "base": 50000.0, "scaling": {
+                "factor": 4.0, "original": 1024, "fast": 32.0, "slow": 1.0}}),
+            "right": {"heads": lh, "dim": ld, "vdim": lv, "tau": 16.0, "decay_rank": rank}}},
+        {"type": "parallel", "mlp": moe, "mixer": {
+            "left": dict(heads, q_temp={"coef": 0.1, "every": 1024}), "right": {"width": rw, "blocks": rb, "conv": taps}}},
+        {"type": "attention", "mlp": moe, "mixer": dict(heads, mask={"size": chunk}, rot={"dims": d, "base": 500000.0, "scaling": {
+            "factor": 8.0, "low": 1.0, "high": 4.0, "original": 1024}})}]
+    return {"architecture": "Saberax", "vocab": DESIGN_VOCAB, "width": w, "norm": {"eps": 1e-6}, "residual_mult": 0.7,
+            "layers": layers * blocks}
+
+
+def feruzen_beside_saberax(size):
+    """As many layers of the same width and heads, attention beside a matrix memory (the recurrent heads with the sizes of the
+    linear attention's) in every layer, and the same feed-forwards with gates."""
+    w, h, g, d, window, chunk, rw, rb, taps, lh, ld, lv, rank, ff, experts, top, eff, groups, sff, blocks = size
+    dense = {"kind": "dense", "ff": ff, "limit": 7.0}
+    moe = {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": eff, "limit": 7.0},
+           "shared": {"ff": sff, "limit": 7.0}}
+    sides = {"type": "parallel", "mixer": {
+        "left": {"heads": h, "kv_heads": g, "dim": d, "vdim": d, "rot": {"dims": d, "base": 500000.0}, "scale": d ** -0.5},
+        "right": {"heads": lh, "dim": ld, "vdim": lv, "gate_cap": 15.0}, "left_scale": 1.0, "right_scale": 1.0}}
+    return {"architecture": "Feruzen", "vocab": DESIGN_VOCAB, "width": w, "norm": {"eps": 1e-6, "groups": 1},
+            "canon": {"taps": taps}, "layers": [dict(sides, mlp=m) for m in (dense, moe, moe)] * blocks}
+
+
+def saberax_arm(args) -> int:
+    """Prefill and decode throughput of the Saberax decoder at sizes of real layers, beside the Feruzen
+    decoder (the closest design the engine has: mixers side by side, attention with options, a recurrence over a
+    matrix state, routed experts with a shared one) with as many layers of the same sizes, and the time the device
+    spends in every kind of kernel call per layer, with the fraction of the roofline for the calls that have one."""
+    import torch
+    from tinyinfer_b200 import Engine, StepEntry
+    pk, pk_kind = peaks()
+    prompt_len, batch, context = args.prefill_tokens, args.batch, args.context
+    warmup = max(args.warmup, 3)
+    out = {"design": "saberax", "beside": "feruzen at equal sizes", "peaks": pk_kind, "prefill_tokens": prompt_len,
+           "decode_batch": batch, "decode_context": context, "dtype": "bf16", "data": "synthetic", "sizes": {}}
+    gen = torch.Generator().manual_seed(0)
+    prompt = torch.randint(0, DESIGN_VOCAB, (prompt_len,), generator=gen).tolist()
+    hbm, tc = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12
+    # float32 multiply-adds on the CUDA cores (128 lanes an SM, the clock's maximum)
+    props = torch.cuda.get_device_properties(0)
+    fp32 = props.multi_processor_count * 128 * 2.0 * getattr(props, "clock_rate", 1965000) * 1e3
+    for key, size in SABERAX_SIZES.items():
+        if args.design_size and key != args.design_size:
+            continue
+        w, h, kvh, d, window, chunk, rw, rb, taps, lh, ld, lv, rank, ff, experts, top, eff, groups, sff, blocks = size
+        n_layers = 3 * blocks
+        res = {}
+        calls = {"saberax": ["attention_options", "heads_prepare_store", "layer_norm", "norm_sum", "causal_conv", "conv_tail_store",
+                             "gated_recurrence", "block_products", "recurrence_rows", "low_rank_decay", "matrix_state", "glu_ffn",
+                             "unary_ffn", "router_choose", "routed_experts", "linear"],
+                 "feruzen": ["attention_options", "qk_rownorm_rope_store", "matrix_state", "causal_conv", "conv_tail_store",
+                             "group_norm", "depth_mix", "add_scaled", "glu_ffn", "router_topk", "routed_experts", "linear"]}
+        for arm, cfg in (("saberax", saberax_config(size)), ("feruzen", feruzen_beside_saberax(size))):
+            engine = Engine(config=cfg, seed=0, dtype="bfloat16", page_size=args.page_size,
+                            num_pages=-(-max(batch * context, prompt_len) // args.page_size) + batch + 2,
+                            max_requests=batch + 1, step_graphs=True)
+            pf_ms = measure_prefill(engine, prompt_len, max(1, min(args.steps, 6)), torch)
+            ms, clocks, launches = measure_decode(engine, batch, context, args.steps, warmup, torch)
+            a = {"prefill_tok_s": round(prompt_len / pf_ms * 1e3), "prefill_ms": round(pf_ms, 3),
+                 "decode_tok_s": round(batch / ms * 1e3, 1), "decode_ms_per_step": round(ms, 4),
+                 "decode_launches_per_step": launches // max(1, args.steps), "clocks": clocks}
+            engine._step_graphs = None
+            engine.ops.fuse_decode_tail = engine.ops.fuse_decode_ffn = engine.ops.pair_few_rows = False   # every call of its own
+            names = calls[arm]
+            for _ in range(2):        # the first eager step sizes the allocator's pool; the second is read
+                spans = timed_ops(engine, names, lambda: engine.step([StepEntry("p", prompt, [prompt_len - 1])]), torch)
+                engine.finish("p")
+            ids = fill_requests(engine, batch, context - 4, torch)
+            for _ in range(2):
+                # a token of its own for every request, so that the routers' choices differ between them
+                dspans = timed_ops(engine, names, lambda: engine.step([StepEntry(r, [1 + 37 * i], [0]) for i, r in enumerate(ids)]), torch)
+            chosen = []
+            inner = engine.ops.routed_experts
+
+            def noting(h_, w_, ids_, *rest, **kw):
+                chosen.append(ids_.clone())
+                return inner(h_, w_, ids_, *rest, **kw)
+
+            engine.ops.routed_experts = noting
+            engine.step([StepEntry(r, [1 + 37 * i], [0]) for i, r in enumerate(ids)])
+            del engine.ops.routed_experts
+            hit = int(chosen[0].unique().numel())          # different experts that a decoding step's first router chose
+            for r in ids:
+                engine.finish(r)
+            a["decode_experts_hit"] = hit
+            a["calls_us"] = {
+                "prompt": {n: [round(x * 1e3, 1) for x in v[:12]] for n, v in spans.items() if not n.startswith("_") and n != "linear"},
+                "decode": {n: [round(x * 1e3, 1) for x in v[:12]] for n, v in dspans.items() if not n.startswith("_") and n != "linear"}}
+            a["per_layer_us"] = {
+                "prompt": {n: round(sum(v) / n_layers * 1e3, 1) for n, v in spans.items() if not n.startswith("_")},
+                "decode": {n: round(sum(v) / n_layers * 1e3, 1) for n, v in dspans.items() if not n.startswith("_")}}
+            seen_all = prompt_len * (prompt_len + 1) / 2
+            att, datt = spans["attention_options"], dspans["attention_options"]
+            st, dst = spans["matrix_state"], dspans["matrix_state"]
+            lin_rows = prompt_len * ((2 * lh * ld + 2 * lh * lv) * 4 + lh * lv * 2.0)
+            cols = (h + 2 * kvh) * d
+
+            def frac(amount, ms_, peak):
+                return round(amount / (ms_ * 1e-3) / peak, 4)
+
+            def product(sp, shape, adds):
+                """The first product with a weight of this shape that adds to its output, or that stores it."""
+                return next((ms_ for ms_, (s, acc) in zip(sp["linear"], sp["_linear_kinds"]) if s == shape and bool(acc) == adds), None)
+
+            roof = a["roofline_frac"] = {
+                "prompt_dense_ffn": frac(2.0 * prompt_len * 3 * w * ff, spans["glu_ffn"][0], tc),
+                "decode_dense_ffn": frac(2.0 * 3 * w * ff, dspans["glu_ffn"][0], hbm)}
+            if arm == "saberax":
+                # calls in layer order: window attention beside linear attention, causal beside the recurrence, chunked
+                seen_window = sum(min(i + 1, window) for i in range(prompt_len))
+                seen_chunk = sum(i % chunk + 1 for i in range(prompt_len))
+                keys = {"window": min(window, context), "causal": context, "chunk": (context - 1) % chunk + 1}
+                for i, (n, seen) in enumerate((("window", seen_window), ("causal", seen_all), ("chunk", seen_chunk))):
+                    roof[f"prompt_{n}_attention"] = frac(4.0 * h * d * seen, att[i], tc)
+                    roof[f"decode_{n}_attention"] = frac(batch * kvh * keys[n] * 2 * d * 2.0, datt[i], hbm)
+                prep, dprep = spans["heads_prepare_store"], dspans["heads_prepare_store"]
+                key_cols = (h + kvh) * d                       # the chunked layer has no value columns, but stores values
+                roof.update({
+                    "prompt_heads_window": frac(prompt_len * cols * (4 + 2.0), prep[0], hbm),
+                    "prompt_heads_causal": frac(prompt_len * cols * (4 + 2.0), prep[1], hbm),
+                    "prompt_heads_chunk": frac(prompt_len * (key_cols * 4 + cols * 2.0), prep[2], hbm),
+                    "decode_heads": frac(batch * cols * (4 + 2.0), dprep[0], hbm),
+                    # experts have two matrices; the shared one runs inside the call
+                    "prompt_experts": frac(2.0 * prompt_len * 2 * w * (top * eff + sff), spans["routed_experts"][0], tc),
+                    "decode_experts": frac(2.0 * 2 * w * (eff * hit + sff), dspans["routed_experts"][0], hbm),
+                    "prompt_linear_attention_fp32": frac(prompt_len * lh * ld * lv * 5.0, st[0], fp32),
+                    "prompt_linear_attention_bytes": frac(lin_rows + prompt_len * lh * ld * 4.0, st[0], hbm),
+                    "decode_linear_attention_state_bytes": frac(batch * lh * ld * lv * 8.0, dst[0], hbm),
+                    "prompt_key_decays_bytes": frac(prompt_len * lh * ld * 4.0, spans["low_rank_decay"][0], hbm),
+                    "prompt_recurrence_bytes": frac(rw * (4 * 4 + 2.0) * prompt_len, spans["recurrence_rows"][0], hbm),
+                    "decode_recurrence_bytes": frac(4.0 * rw * (rw // rb) + batch * rw * 18.0, dspans["gated_recurrence"][0], hbm),
+                    "prompt_convolution": frac(prompt_len * rw * 8.0, spans["causal_conv"][0], hbm),
+                    "prompt_norm": frac(prompt_len * w * (4 + 2.0), spans["layer_norm"][0], hbm),
+                    "decode_norm": frac(batch * w * (4 + 2.0), dspans["layer_norm"][0], hbm),
+                    # two rows in, the residual in and out, the normed row out
+                    "prompt_normed_sides": frac(prompt_len * w * (4 + 4 + 8 + 2.0), spans["norm_sum"][0], hbm),
+                    "decode_normed_sides": frac(batch * w * (4 + 4 + 8 + 2.0), dspans["norm_sum"][0], hbm),
+                    # the sides' first products as one, and a closing product that stores (Feruzen's adds)
+                    "prompt_side_product": frac(2.0 * prompt_len * w * h * d, product(spans, (w, h * d), False), tc),
+                    "decode_side_product": frac(2.0 * w * h * d, product(dspans, (w, h * d), False), hbm),
+                    "prompt_router": frac(prompt_len * (experts * 4 + top * 8.0), spans["router_choose"][0], hbm)})
+            else:
+                roof.update({
+                    "prompt_attention": frac(4.0 * h * d * seen_all, att[0], tc),
+                    "decode_attention": frac(batch * kvh * context * 2 * d * 2.0, datt[0], hbm),
+                    "prompt_heads": frac(prompt_len * cols * (4 + 2.0), spans["qk_rownorm_rope_store"][0], hbm),
+                    "decode_heads": frac(batch * cols * (4 + 2.0), dspans["qk_rownorm_rope_store"][0], hbm),
+                    "prompt_experts": frac(2.0 * prompt_len * top * 3 * w * eff, spans["routed_experts"][0], tc),
+                    "decode_experts": frac(2.0 * 3 * w * eff * hit, dspans["routed_experts"][0], hbm),
+                    "prompt_matrix_memory_fp32": frac(prompt_len * lh * ld * (lv + 1) * 5.0, st[0], fp32),
+                    "prompt_matrix_memory_bytes": frac(lin_rows + prompt_len * 2 * lh * 4.0, st[0], hbm),
+                    "decode_matrix_memory_state_bytes": frac(batch * lh * ld * (lv + 1) * 8.0, dst[0], hbm),
+                    "prompt_convolution": frac(prompt_len * w * (4 + 2.0), spans["causal_conv"][0], hbm),
+                    "prompt_norm_added": frac(prompt_len * w * (4 + 4 + 4.0), spans["group_norm"][0], hbm),
+                    "decode_norm_added": frac(batch * w * (4 + 4 + 4.0), dspans["group_norm"][0], hbm),
+                    "prompt_sum_of_sides": frac(prompt_len * w * (4 + 4 + 8.0), spans["add_scaled"][0], hbm),
+                    "prompt_side_product": frac(2.0 * prompt_len * w * h * d, product(spans, (w, h * d), True), tc),
+                    "decode_side_product": frac(2.0 * w * h * d, product(dspans, (w, h * d), True), hbm),
+                    "prompt_router": frac(prompt_len * (experts * 4 + top * 8.0), spans["router_topk"][0], hbm)})
+            res[arm] = a
+            del engine
+            torch.cuda.empty_cache()
+        out["sizes"][key] = {"width": w, "heads": h, "kv_heads": kvh, "head_dim": d, "window": window, "chunk": chunk,
+                             "recurrence": [rw, rb], "taps": taps, "linear_attention": [lh, ld, lv], "decay_rank": rank, "ff": ff,
+                             "experts": experts, "top": top, "expert_ff": eff, "groups": list(groups), "shared_ff": sff,
+                             "layers": n_layers, **res}
+    print(json.dumps(out))
+    return 0
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1295,9 +1487,9 @@ def main() -> int:
                     help="with --only mixed: the number of decoding requests beside the 512-token portion")
     ap.add_argument("--attention-in-turn", action="store_true",
                     help="with --only mixed: flash-decoding behind the prompt attention kernel, not beside it")
-    ap.add_argument("--design", choices=["kagorax", "ruvuvik", "feruzen", "nekorax", "vametar"], default=None,
-                    help="set this decoder beside the closest one the engine has (Qwen3; for feruzen and nekorax: Ruvuvik; for vametar: Feruzen) at equal sizes instead of the default run")
-    ap.add_argument("--design-size", choices=sorted(set(DESIGN_SIZES) | set(RUVUVIK_SIZES) | set(FERUZEN_SIZES) | set(NEKORAX_SIZES) | set(VAMETAR_SIZES)), default=None,
+    ap.add_argument("--design", choices=["kagorax", "ruvuvik", "feruzen", "nekorax", "vametar", "saberax"], default=None,
+                    help="set this decoder beside the closest one the engine has (Qwen3; for feruzen and nekorax: Ruvuvik; for vametar and saberax: Feruzen) at equal sizes instead of the default run")
+    ap.add_argument("--design-size", choices=sorted(set(DESIGN_SIZES) | set(RUVUVIK_SIZES) | set(FERUZEN_SIZES) | set(NEKORAX_SIZES) | set(VAMETAR_SIZES) | set(SABERAX_SIZES)), default=None,
                     help="one of the sizes only")
     ap.add_argument("--only", choices=["decode", "prefill", "chains", "mixed"], default=None,
                     help="run one part only and print a short line (for profiling small cases)")
@@ -1317,6 +1509,8 @@ def main() -> int:
         return nekorax_arm(args)
     if args.design == "vametar":
         return vametar_arm(args)
+    if args.design == "saberax":
+        return saberax_arm(args)
     if args.design:
         return design_arm(args)
 
