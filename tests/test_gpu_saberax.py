@@ -285,7 +285,7 @@ def _part(ops, category, spec, w):
 @pytest.mark.parametrize("mlp", [moe(12, 3, 24, 1.7, groups=(3, 2), shared=40), moe(8, 2, 16, 2.5, groups=(2, 1)), moe(4, 4, 12, 1.0),
                                  moe(5, 1, 9, 3.0, groups=(1, 1), shared=7), moe(16, 4, 64, 2.0, groups=(4, 2), shared=128),
                                  moe(3, 2, 32, 1.5, shared=4096), dense(40), dense(192)])
-@pytest.mark.parametrize("t", [1, 7, 150, 700])      # 150 and 700 rows: the grouped products on the tensor cores
+@pytest.mark.parametrize("t", [1, 7, 60, 150, 700])  # 60: a shared expert beside the router; 150, 700: grouped products
 def test_each_feed_forward_alone(ops, mlp, t, dtype):
     from tinyinfer_b200.config import saberax
     from tinyinfer_b200.parts.base import GatedSum

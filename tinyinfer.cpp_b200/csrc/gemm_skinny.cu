@@ -277,16 +277,16 @@ extern "C" int ti_gemm_skinny_gated(const void* a, const void* w, float* c, int 
 }
 
 // Two products of m rows in one launch: the first stores its float32 rows into c, or (glu_kind >= 0)
-// its gated activation over strips of 8 and 8 into out_act; the second stores a2 w2^T into c2.
+// its gated activation over strips of 8 and 8, or an activation of one value, into out_act; the second stores a2 w2^T into c2.
 extern "C" int ti_gemm_skinny_pair(const void* a, const void* w, float* c, void* out_act, int m, int n, int k, int lda,
                                    int ldw, int ldc, int ld_act, int glu_kind, float glu_limit, float glu_alpha,
                                    const void* a2, const void* w2, float* c2, int n2, int k2, int lda2, int ldw2, int ldc2,
                                    void* stream) {
     if (m == 0 || n == 0 || n2 == 0) return 0;
-    TI_REQUIRE(glu_kind <= GLU_GELU_TANH, "gemm_skinny_pair: activation %d", glu_kind);
+    TI_REQUIRE(glu_kind <= GLU_GELU_TANH || glu_kind == ACT_RELU2, "gemm_skinny_pair: activation %d", glu_kind);
     TI_REQUIRE(ti_gemm_skinny_supported(m, n2, k2, lda2, ldw2) && (uintptr_t)a2 % 16 == 0 && (uintptr_t)w2 % 16 == 0,
                "gemm_skinny_pair: the second product's operands");
-    return skinny(a, w, c, out_act, m, n, k, lda, ldw, ldc, ld_act, glu_kind < 0 ? MODE_STORE : MODE_SWIGLU,
+    return skinny(a, w, c, out_act, m, n, k, lda, ldw, ldc, ld_act, glu_kind < 0 ? MODE_STORE : act_is_gated(glu_kind) ? MODE_SWIGLU : MODE_UNARY,
                   glu_kind < 0 ? GLU_SILU : glu_kind, glu_limit, glu_alpha, stream, AddGate{nullptr, 0, nullptr, 1.0f},
                   SecondProduct{(const bf16*)a2, (const bf16*)w2, c2, n2, k2, lda2, ldw2, ldc2, 0});
 }

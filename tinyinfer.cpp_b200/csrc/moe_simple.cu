@@ -41,7 +41,7 @@ __device__ __forceinline__ float sigmoidf_(float z) { return 1.0f / (1.0f + expf
 // aligned go eight elements a load (a warp then asks for 512 contiguous bytes of a weight row at
 // once, instead of 64); everything else one element at a time.
 template <typename TA, typename TW>
-__device__ __forceinline__ void lane_dots(const TA* __restrict__ x, const TW* __restrict__ a, const TW* __restrict__ b,
+__device__ __forceinline__ void lane_dots(const TA* x, const TW* __restrict__ a, const TW* __restrict__ b,
                                           int n, int lane, float& ra, float& rb) {
     ra = rb = 0.0f;
     if constexpr (sizeof(TA) == 2 && sizeof(TW) == 2) {
@@ -150,6 +150,8 @@ router_choose_kernel(const float* logits, int stride, int num_tokens, int total,
                      int normalize, float factor, int* __restrict__ ids, float* __restrict__ weights) {
     __shared__ float choice[WARPS][MAX_ROUTED];
     __shared__ float group_best[WARPS][MAX_GROUPS];
+    pdl_launch();
+    pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x * WARPS + warp;
     if (t >= num_tokens) return;
@@ -223,12 +225,13 @@ router_choose_kernel(const float* logits, int stride, int num_tokens, int total,
 // one warp per output element f of one (token, slot)
 template <typename TA, typename TW>
 __global__ void __launch_bounds__(WARPS * 32)
-moe_gate_up_simple_kernel(const TA* __restrict__ h, int h_stride, const TW* __restrict__ w_gate_up,
-                          int interleaved, const int* __restrict__ ids,
-                          const float* __restrict__ weights, int top, int width, int ff,
+moe_gate_up_simple_kernel(const TA* h, int h_stride, const TW* __restrict__ w_gate_up,
+                          int interleaved, const int* ids, const float* weights, int top, int width, int ff,
                           TA* __restrict__ y, int n_pairs, const TW* __restrict__ shared_gate_up,
                           int shared_interleaved, int shared_ff, TA* __restrict__ y_shared,
                           int act, float act_limit, float act_alpha, int experts) {
+    pdl_launch();
+    pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     int ts = blockIdx.x;                              // token * top + slot; behind the pairs: a token's shared expert
     const int f = blockIdx.y * WARPS + warp;
@@ -271,12 +274,14 @@ moe_gate_up_simple_kernel(const TA* __restrict__ h, int h_stride, const TW* __re
 
 template <typename TA, typename TW>
 __global__ void __launch_bounds__(WARPS * 32)
-moe_down_simple_kernel(const TA* __restrict__ y, const TW* __restrict__ w_down,
-                       const int* __restrict__ ids, int top, int width, int ff,
-                       float* __restrict__ out, int out_stride, const TA* __restrict__ y_shared,
-                       const TW* __restrict__ w_shared_down, const float* __restrict__ shared_gate,
-                       int shared_ff, int experts, const TA* __restrict__ h, int h_stride,
-                       const float* __restrict__ weights, float shared_factor) {
+moe_down_simple_kernel(const TA* y, const TW* __restrict__ w_down,
+                       const int* ids, int top, int width, int ff,
+                       float* out, int out_stride, const TA* y_shared,
+                       const TW* __restrict__ w_shared_down, const float* shared_gate,
+                       int shared_ff, int experts, const TA* h, int h_stride,
+                       const float* weights, float shared_factor) {
+    pdl_launch();
+    pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x;
     const int n = blockIdx.y * WARPS + warp;
@@ -348,7 +353,7 @@ extern "C" int ti_router_choose(const float* logits, int stride, int num_tokens,
     TI_REQUIRE(best_of == 1 || best_of == 2, "router_choose: a group's value is its largest or the sum of its two largest");
     TI_REQUIRE(top >= 1 && top <= MAX_TOP && top <= total / groups * keep,
                "router_choose: %d of %d outputs cannot be chosen", top, total / groups * keep);
-    router_choose_kernel<<<(num_tokens + WARPS - 1) / WARPS, WARPS * 32, 0, (cudaStream_t)stream>>>(
+    ti_launch_pdl(router_choose_kernel, dim3((num_tokens + WARPS - 1) / WARPS), dim3(WARPS * 32), 0, (cudaStream_t)stream,
         logits, stride, num_tokens, total, top, correction, groups, keep, sigmoid, best_of, normalize, factor, ids, weights);
     return ti_check_launch("router_choose");
 }
@@ -366,7 +371,7 @@ extern "C" int ti_moe_gate_up_simple(const void* h, int act_dtype, int h_stride,
     dim3 grid(num_tokens * top + (shared ? num_tokens : 0), (most + WARPS - 1) / WARPS);
     cudaStream_t s = (cudaStream_t)stream;
 #define CALL(TA, TW)                                                                         \
-    moe_gate_up_simple_kernel<TA, TW><<<grid, WARPS * 32, 0, s>>>(                            \
+    ti_launch_pdl(moe_gate_up_simple_kernel<TA, TW>, grid, dim3(WARPS * 32), 0, s,            \
         (const TA*)h, h_stride, (const TW*)w_gate_up, interleaved, ids, weights, top, width, ff, (TA*)y, \
         num_tokens * top, (const TW*)shared_gate_up, shared_interleaved, shared_ff, (TA*)y_shared, \
         act, act_limit, act_alpha, experts)
@@ -385,7 +390,7 @@ extern "C" int ti_moe_down_simple(const void* y, int act_dtype, const void* w_do
     dim3 grid(num_tokens, (width + WARPS - 1) / WARPS);
     cudaStream_t s = (cudaStream_t)stream;
 #define CALL(TA, TW)                                                                         \
-    moe_down_simple_kernel<TA, TW><<<grid, WARPS * 32, 0, s>>>(                               \
+    ti_launch_pdl(moe_down_simple_kernel<TA, TW>, grid, dim3(WARPS * 32), 0, s,               \
         (const TA*)y, (const TW*)w_down, ids, top, width, ff, out, out_stride, (const TA*)y_shared, \
         (const TW*)w_shared_down, shared_gate, shared_ff, experts, (const TA*)h, h_stride, weights, shared_factor)
     TI_DISPATCH_AW(act_dtype, w_dtype, CALL)

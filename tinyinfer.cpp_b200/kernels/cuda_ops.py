@@ -140,6 +140,8 @@ class CudaOps(MixerOps, StateOps):
         self.grouped_experts_from = 128       # (token, slot) pairs from which the experts run as grouped products
         self.tcgen05_experts_from = 1024      # ... and from which those products run on tcgen05
         self.shared_rides_to = 1 << 17        # elements of a shared expert's matrix up to which it rides along
+        # ... and for experts without a gate (bfloat16), tokens times elements: what the riding form reads from L2
+        self.shared_rides_reads = 1 << 23
         self._counters = None
         self.use_tc_attention = True      # tcgen05 prompt attention where the shape allows
         self.use_2sm_gemm = True          # pairs of SMs for products with enough 256 x 256 tiles
@@ -664,6 +666,9 @@ class CudaOps(MixerOps, StateOps):
               and h.stride(1) == w.stride(1) == out.stride(1) == 1, "linear_unary: shapes do not agree")
         if h.dtype == w.dtype == torch.bfloat16 and h.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0:
             if self.bf16.ti_gemm_skinny_supported(m, n, k, h.stride(0), w.stride(0)):
+                if self._launch_pair(h, w, None, out, (UNARY_KINDS[kind], 0.0, 0.0)):
+                    return
+                self.flush()
                 self._ok(self.bf16.ti_gemm_skinny_unary(h.data_ptr(), w.data_ptr(), out.data_ptr(), m, n, k, h.stride(0),
                                                         w.stride(0), out.stride(0), UNARY_KINDS[kind], self._stream()),
                          self.bf16)
@@ -1263,16 +1268,43 @@ class CudaOps(MixerOps, StateOps):
         activation, ``(kind, limit, alpha)`` as ``glu_rows`` takes them; the pair's weight then
         scales the expert's output, residual[t] += w Wdown_e act(g, u), and there is no ``shared``.
         Experts without a gate (``pack_experts(None, ...)``) take an activation of one value, residual[t] += w
-        Wdown_e act(u); their ``shared`` is ``(w_up, w_down, factor)``, residual[t] += factor Wdown act(Wup h[t]).
+        Wdown_e act(u); their ``shared`` is ``(w_up, w_down, factor)``, residual[t] += factor Wdown act(Wup h[t])
+        (``router_beside_shared`` may have put ``act(Wup h)`` behind the three).
         ``identity``: an index at or behind the number of stacked experts names an identity expert,
         whose output is the token's input, residual[t] += w h[t]."""
         self._routed(h, w, ids, weights, residual, shared, act, identity)
 
+    def _unary_shared_rides(self, h, shared) -> bool:
+        """Whether a shared expert without a gate runs inside the experts' two launches (of few tokens)."""
+        most = shared[1].shape[1] * shared[1].shape[0]
+        if h.dtype != torch.bfloat16:                # a float32 row's bits must not depend on the step around it
+            return most <= self.shared_rides_to
+        return h.shape[0] * most <= self.shared_rides_reads
+
+    def router_beside_shared(self, h, w_router, logits, top, shared, act):
+        """``logits = h w_router^T``, and, where few rows allow it, the first product of the shared expert ``shared``
+        (as ``routed_experts`` takes it, of experts without a gate) in the same launch.  Returns ``shared``, with
+        the activations of that product behind it if it has run."""
+        w_up = shared[0]
+        pairs = h.shape[0] * top
+        grouped = (self.grouped_experts_from is not None and pairs >= self.grouped_experts_from)
+        if grouped or self._unary_shared_rides(h, shared) or not self._pairable(h, w_up):
+            self.linear(h, w_router, logits)
+            return shared
+        self.linear(h, w_router, logits, may_pair=True)
+        y = torch.empty((h.shape[0], w_up.shape[0]), dtype=h.dtype, device=h.device)
+        self.linear_unary(h, w_up, act[0], y)
+        return (*shared, y)
+
     def _shared_expert(self, h, shared, residual, act=None):
-        w_gate_up, w_down, gate = shared
+        w_gate_up, w_down, gate = shared[:3]
         if not isinstance(gate, torch.Tensor):       # no gate of either sort: one factor for all tokens
             from ..parts.base import GatedSum
-            self.unary_ffn(h, w_gate_up, w_down, residual if gate == 1.0 else GatedSum(residual, None, None, gate), act[0])
+            target = residual if gate == 1.0 else GatedSum(residual, None, None, gate)
+            if len(shared) > 3:                      # its first product has run already
+                self.linear(shared[3], w_down, target, accumulate=True)
+            else:
+                self.unary_ffn(h, w_gate_up, w_down, target, act[0])
             return
         y = torch.empty((h.shape[0], w_down.shape[1]), dtype=h.dtype, device=h.device)
         self.gate_up_swiglu(h, w_gate_up, y)
@@ -1357,8 +1389,8 @@ class CudaOps(MixerOps, StateOps):
         # batch 8: 5,784 -> 5,277 tok/s with a shared expert of 2,048 x 4,096 riding along)
         ride = (shared is not None and shared[0].dtype == gate_up.dtype and shared[1].dtype == gate_up.dtype
                 and shared[0].is_contiguous() and shared[1].is_contiguous()
-                and (not gated or shared[2].dtype == torch.float32)
-                and shared[1].shape[1] * width <= self.shared_rides_to)
+                and (self._unary_shared_rides(h, shared) and len(shared) == 3 if not gated else
+                     shared[2].dtype == torch.float32 and shared[1].shape[1] * width <= self.shared_rides_to))
         y_sh = sgu = sdown = sgate = None
         s_ff = s_inter = 0
         s_factor = 1.0

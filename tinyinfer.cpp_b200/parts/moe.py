@@ -134,7 +134,12 @@ class RoutedExperts(Part):
         t = h.shape[0]
         residual, factor = residual_and_factor(residual)     # a factor on the sublayer: on the weights, and on the shared expert
         logits = torch.empty((t, self.w_router.shape[0]), dtype=torch.float32, device=h.device)
-        ops.linear(h, self.w_router, logits)
+        shared = None
+        if not self.gated and self.shared_size is not None:
+            shared = ops.router_beside_shared(h, self.w_router, logits, self.top,
+                                              (self.w_shared_gate_up, self.w_shared_down, factor), self.activation)
+        else:
+            ops.linear(h, self.w_router, logits)
         ids = torch.empty((t, self.top), dtype=torch.int32, device=h.device)
         weights = torch.empty((t, self.top), dtype=torch.float32, device=h.device)
         shared_gate = None
@@ -150,7 +155,6 @@ class RoutedExperts(Part):
         else:
             ops.router_topk(logits, self.experts, self.top, ids, weights, shared_gate, softmax=self.router == "softmax")
         if not self.gated:
-            shared = None if self.shared_size is None else (self.w_shared_gate_up, self.w_shared_down, factor)
             ops.routed_experts(h, self.w_experts, ids, weights, residual, shared, act=self.activation)
             return
         shared = None
