@@ -10,8 +10,8 @@
 // then keys and values go into the token's page and queries into q_out.  `values_from_keys`: there are no value
 // columns, a value head is the key head's columns (with their bias) as they are; dv = dk.
 //
-// A block takes one token, whose cosines and sines it makes once, and a share of its heads; a head belongs to 4 to 32
-// lanes of a warp, which hold it in registers as units of four elements (two pairs), so it is read once.  Sizes
+// A block takes one token, whose cosines and sines it makes once, and a share of its heads; a head belongs to 8, 16 or
+// 32 lanes of a warp, which hold it in registers as units of four elements (two pairs), so it is read once.  Sizes
 // that do not fall into such units take a kernel with a warp per head and a pass per norm.  All arithmetic is
 // float32; a head's bits depend on its row alone.
 #include "common.cuh"
@@ -69,8 +69,9 @@ __device__ __forceinline__ TC* token_page(const Heads& p, int t, int pos, TC* pa
     return pages + (size_t)page * p.num_kv_heads * p.page_size * (p.dk + p.dv);
 }
 
-__device__ __forceinline__ float group_sum(float v, int lanes) {
-    for (int o = lanes >> 1; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+template <int LANES> __device__ __forceinline__ float group_sum(float v) {
+#pragma unroll
+    for (int o = LANES / 2; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
     return v;
 }
 
@@ -105,12 +106,77 @@ __device__ __forceinline__ void store_unit(T* p, int u, bool turned, int halves,
 __device__ __forceinline__ float squares(float4 v) { return fmaf(v.w, v.w, fmaf(v.z, v.z, fmaf(v.y, v.y, v.x * v.x))); }
 __device__ __forceinline__ void times(float4& v, float f) { v.x *= f; v.y *= f; v.z *= f; v.w *= f; }
 
-// `lanes` (a power of two up to 32) lanes a head, NU units a lane
-template <typename TQ, typename TC, int NU>
+// What a head of KIND goes through between its row and its destination.  LANES lanes hold it, NU units a lane.
+template <int KIND, int LANES, int NU, typename T>
+__device__ __forceinline__ void prepare_head(const Heads& p, const float* row, int column, const float2* cs, float factor,
+                                             int lane, bool live, T* dst) {
+    const int n = KIND == ITEM_VALUE ? p.dv : p.dk;
+    const int units = n >> 2, turned_units = KIND == ITEM_VALUE ? 0 : p.rot >> 2, half = p.rot >> 1;
+    const float* src = row + column;
+    float4 v[NU];
+    float ss = 0.0f;
+#pragma unroll
+    for (int j = 0; j < NU; ++j) {
+        const int u = lane + LANES * j;
+        v[j] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (!live || u >= units) continue;
+        const bool turned = u < turned_units;
+        v[j] = load_unit(src, u, turned, p.halves, half);
+        if (p.bias) {
+            const float4 b = load_unit(p.bias + column, u, turned, p.halves, half);
+            v[j].x += b.x; v[j].y += b.y; v[j].z += b.z; v[j].w += b.w;
+        }
+        if (KIND != ITEM_VALUE) ss += squares(v[j]);
+    }
+    if (KIND != ITEM_VALUE) {
+        const float mean_of = 1.0f / (float)n;
+        float last = KIND == ITEM_QUERY ? factor : 1.0f;
+        if (p.pre_norm) {
+            const float inv = rsqrtf(fmaf(group_sum<LANES>(ss), mean_of, p.eps));
+            const float* w = KIND == ITEM_QUERY ? p.q_weight : p.k_weight;
+            if (w) {
+#pragma unroll
+                for (int j = 0; j < NU; ++j) {
+                    const int u = lane + LANES * j;
+                    if (u >= units) continue;
+                    const float4 g = load_unit(w, u, u < turned_units, p.halves, half);
+                    v[j].x *= inv * g.x; v[j].y *= inv * g.y; v[j].z *= inv * g.z; v[j].w *= inv * g.w;
+                }
+            } else {
+#pragma unroll
+                for (int j = 0; j < NU; ++j) times(v[j], inv);
+            }
+        }
+#pragma unroll
+        for (int j = 0; j < NU; ++j) {
+            const int u = lane + LANES * j;
+            if (u >= turned_units) continue;
+            const float4 f = *reinterpret_cast<const float4*>(cs + 2 * u);     // two pairs' (cosine, sine)
+            v[j] = make_float4(v[j].x * f.x - v[j].z * f.y, v[j].y * f.z - v[j].w * f.w,
+                               v[j].z * f.x + v[j].x * f.y, v[j].w * f.z + v[j].y * f.w);
+        }
+        if (p.post_norm) {
+            float sq = 0.0f;
+#pragma unroll
+            for (int j = 0; j < NU; ++j) sq += squares(v[j]);
+            last *= rsqrtf(fmaf(group_sum<LANES>(sq), mean_of, p.eps));
+        }
+#pragma unroll
+        for (int j = 0; j < NU; ++j) times(v[j], last);
+    }
+    if (!live || dst == nullptr) return;
+#pragma unroll
+    for (int j = 0; j < NU; ++j) {
+        const int u = lane + LANES * j;
+        if (u < units) store_unit<T>(dst, u, u < turned_units, p.halves, half, v[j]);
+    }
+}
+
+// LANES lanes of a warp a head, NU units a lane
+template <typename TQ, typename TC, int LANES, int NU>
 __global__ void __launch_bounds__(THREADS)
-heads_prepare_store_kernel(const Heads p, int lanes, TC* __restrict__ pages, TQ* __restrict__ q_out,
-                           int* __restrict__ status) {
-    extern __shared__ float2 cs[];
+heads_prepare_store_kernel(const Heads p, TC* __restrict__ pages, TQ* __restrict__ q_out, int* __restrict__ status) {
+    extern __shared__ __align__(16) float2 cs[];
     const int t = blockIdx.x, pos = p.positions[t];
     pdl_launch();
     fill_table(cs, p, (float)pos);                        // of the step's positions: before the wait
@@ -119,72 +185,33 @@ heads_prepare_store_kernel(const Heads p, int lanes, TC* __restrict__ pages, TQ*
     __syncthreads();
     pdl_wait();
     const float* row = p.proj + (size_t)t * p.stride;
-    const int half = p.rot >> 1, slot = pos % p.page_size;
-    const int lane = threadIdx.x & (lanes - 1), per_block = THREADS / lanes;
+    const int slot = pos % p.page_size, nq = p.num_heads * p.dk, nk = p.num_kv_heads * p.dk;
+    constexpr int PER_BLOCK = THREADS / LANES;
+    const int lane = threadIdx.x % LANES, mine = blockIdx.y * PER_BLOCK + threadIdx.x / LANES, step = gridDim.y * PER_BLOCK;
     const int items = p.num_heads + (p.write_kv ? 2 * p.num_kv_heads : 0);
-    for (int first = blockIdx.y * per_block; first < items; first += gridDim.y * per_block) {
-        const int at = first + threadIdx.x / lanes;       // the whole warp walks on together: it sums in groups
-        const bool live = at < items;
-        const Item it = item_of(p, live ? at : 0);
-        const int units = live ? it.n >> 2 : 0, turned_units = it.kind == ITEM_VALUE ? 0 : p.rot >> 2;
-        float4 v[NU];
-        float ss = 0.0f;
-#pragma unroll
-        for (int j = 0; j < NU; ++j) {
-            const int u = lane + lanes * j;
-            v[j] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-            if (u >= units) continue;
-            const bool turned = u < turned_units;
-            v[j] = load_unit(row + it.column, u, turned, p.halves, half);
-            if (p.bias) {
-                const float4 b = load_unit(p.bias + it.column, u, turned, p.halves, half);
-                v[j].x += b.x; v[j].y += b.y; v[j].z += b.z; v[j].w += b.w;
-            }
-            ss += squares(v[j]);
+    // a warp's groups walk on together (they sum in groups): queries, then keys, then values; `at` counts through all
+    const int warp_first = mine - (threadIdx.x % 32) / LANES;
+    for (int first = warp_first, at = mine; first < items; first += step, at += step) {
+        // a warp that holds heads of two kinds takes each kind's path once
+        const int last = first + 32 / LANES - 1, k0 = p.num_heads, v0 = p.num_heads + p.num_kv_heads;
+        if (first < k0) {
+            const bool live = at < k0;
+            prepare_head<ITEM_QUERY, LANES, NU, TQ>(p, row, at * p.dk, cs, factor, lane, live,
+                                                    q_out + ((size_t)t * p.num_heads + at) * p.dk);
         }
-        if (p.pre_norm) {
-            const float inv = 1.0f / sqrtf(group_sum(ss, lanes) / (float)it.n + p.eps);
-            const float* w = it.kind == ITEM_QUERY ? p.q_weight : p.k_weight;
-            if (it.kind != ITEM_VALUE) {
-#pragma unroll
-                for (int j = 0; j < NU; ++j) {
-                    const int u = lane + lanes * j;
-                    if (u >= units) continue;
-                    times(v[j], inv);
-                    if (w) {
-                        const float4 g = load_unit(w, u, u < turned_units, p.halves, half);
-                        v[j].x *= g.x; v[j].y *= g.y; v[j].z *= g.z; v[j].w *= g.w;
-                    }
-                }
-            }
+        if (!p.write_kv) continue;
+        if (last >= k0 && first < v0) {
+            const bool live = at >= k0 && at < v0;
+            const int g = at - k0;
+            prepare_head<ITEM_KEY, LANES, NU, TC>(p, row, nq + g * p.dk, cs, factor, lane, live,
+                                                  page ? page + ((size_t)g * p.page_size + slot) * p.dk : nullptr);
         }
-        ss = 0.0f;
-#pragma unroll
-        for (int j = 0; j < NU; ++j) {
-            const int u = lane + lanes * j;
-            if (u < turned_units && u < units) {
-                const float2 f = cs[2 * u], g = cs[2 * u + 1];
-                v[j] = make_float4(v[j].x * f.x - v[j].z * f.y, v[j].y * g.x - v[j].w * g.y,
-                                   v[j].z * f.x + v[j].x * f.y, v[j].w * g.x + v[j].y * g.y);
-            }
-            ss += squares(v[j]);
-        }
-        float last = it.kind == ITEM_QUERY ? factor : 1.0f;
-        if (p.post_norm) {
-            const float inv = 1.0f / sqrtf(group_sum(ss, lanes) / (float)it.n + p.eps);
-            if (it.kind != ITEM_VALUE) last *= inv;
-        }
-        if (!live || (it.kind != ITEM_QUERY && page == nullptr)) continue;
-#pragma unroll
-        for (int j = 0; j < NU; ++j) {
-            const int u = lane + lanes * j;
-            if (u >= units) continue;
-            const bool turned = u < turned_units;
-            times(v[j], last);
-            if (it.kind == ITEM_QUERY)
-                store_unit<TQ>(q_out + ((size_t)t * p.num_heads + it.head) * p.dk, u, turned, p.halves, half, v[j]);
-            else
-                store_unit<TC>(page_head<TQ, TC>(p, it, page, slot), u, turned, p.halves, half, v[j]);
+        if (last >= v0) {
+            const bool live = at >= v0 && at < items;
+            const int g = at - v0;
+            TC* base = page ? page + (size_t)p.num_kv_heads * p.page_size * p.dk : nullptr;
+            prepare_head<ITEM_VALUE, LANES, NU, TC>(p, row, p.values_from_keys ? nq + g * p.dk : nq + nk + g * p.dv, cs, factor,
+                                                    lane, live, base ? base + ((size_t)g * p.page_size + slot) * p.dv : nullptr);
         }
     }
 }
@@ -268,20 +295,21 @@ extern "C" int ti_heads_prepare_store(const float* proj, int stride, const float
     const bool units = dk % 4 == 0 && dv % 4 == 0 && rot % 4 == 0 && stride % 4 == 0 && widest <= 512 && multiple16(proj) &&
                        multiple16(bias) && multiple16(q_weight) && multiple16(k_weight) && multiple16(pages) &&
                        multiple16(q_out);
-    int lanes = 4;
+    int lanes = 8;
     while (lanes < 32 && lanes * 4 < widest) lanes *= 2;
-    const int nu = (widest / 4 + lanes - 1) / lanes;
+    const int nu = (widest / 4 + 31) / 32;
     const int items = num_heads + (write_kv ? 2 * num_kv_heads : 0), per_block = THREADS / lanes;
     // few tokens: a token's heads over several blocks
     const int gy = num_tokens >= 256 ? 1 : (items + per_block - 1) / per_block;
     cudaStream_t s = (cudaStream_t)stream;
-#define LAUNCH(TQ, TC, NU)                                                                                       \
-    ti_launch_pdl(heads_prepare_store_kernel<TQ, TC, NU>, dim3(num_tokens, gy), dim3(THREADS), smem, s, p, lanes,   \
+#define LAUNCH(TQ, TC, LANES, NU)                                                                                \
+    ti_launch_pdl(heads_prepare_store_kernel<TQ, TC, LANES, NU>, dim3(num_tokens, gy), dim3(THREADS), smem, s, p,   \
                   (TC*)pages, (TQ*)q_out, status)
 #define CALL(TQ, TC)                                                                                             \
     if (!units) ti_launch_pdl(heads_prepare_any_kernel<TQ, TC>, dim3(num_tokens), dim3(THREADS), smem, s, p,        \
                               (TC*)pages, (TQ*)q_out, status);                                                   \
-    else if (nu <= 1) LAUNCH(TQ, TC, 1); else if (nu <= 2) LAUNCH(TQ, TC, 2); else LAUNCH(TQ, TC, 4)
+    else if (lanes <= 8) LAUNCH(TQ, TC, 8, 1); else if (lanes <= 16) LAUNCH(TQ, TC, 16, 1);                       \
+    else if (nu <= 1) LAUNCH(TQ, TC, 32, 1); else if (nu <= 2) LAUNCH(TQ, TC, 32, 2); else LAUNCH(TQ, TC, 32, 4)
     if (q_dtype == TI_F32 && cache_dtype == TI_F32) { CALL(float, float); }
     else if (q_dtype == TI_BF16 && cache_dtype == TI_BF16) { CALL(bf16, bf16); }
     else if (q_dtype == TI_F32 && cache_dtype == TI_BF16) { CALL(float, bf16); }

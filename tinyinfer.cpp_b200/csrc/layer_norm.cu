@@ -212,7 +212,7 @@ extern "C" int ti_norm_sum_rows(const float* a, const float* b, const float* wa,
     TI_REQUIRE(out == nullptr || (then_w != nullptr && then_b != nullptr), "norm_sum_rows: the norm behind the sum");
     cudaStream_t s = (cudaStream_t)stream;
     bool warp;
-    const bool regs = form(n, num_rows, out_dtype == TI_F32, 1024, warp) && res_stride % 4 == 0 && aligned16(a) &&
+    const bool regs = form(n, num_rows, out_dtype == TI_F32, 512, warp) && res_stride % 4 == 0 && aligned16(a) &&
                       aligned16(b) && aligned16(wa) && aligned16(wb) && aligned16(residual) && aligned16(then_w) &&
                       aligned16(then_b) && aligned16(out);
     const int quads = (n / 4 + (warp ? 31 : THREADS - 1)) / (warp ? 32 : THREADS);
@@ -223,7 +223,7 @@ extern "C" int ti_norm_sum_rows(const float* a, const float* b, const float* wa,
 #define CALL(TO)                                                                                                    \
     if (!regs) ti_launch_pdl(norm_sum_any_kernel<TO>, dim3(num_rows), dim3(THREADS), 0, s, a, b, wa, wb, eps, scale,     \
                              residual, res_stride, n, then, (TO*)out);                                              \
-    else if (warp) { if (quads <= 4) LAUNCH(TO, 32, 4); else LAUNCH(TO, 32, 8); }                                   \
+    else if (warp) LAUNCH(TO, 32, 4);                                                                               \
     else { if (quads <= 1) LAUNCH(TO, 256, 1); else if (quads <= 2) LAUNCH(TO, 256, 2);                              \
            else if (quads <= 4) LAUNCH(TO, 256, 4); else LAUNCH(TO, 256, 8); }
     if (out_dtype == TI_F32) { CALL(float) } else { CALL(bf16) }
